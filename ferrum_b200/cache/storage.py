@@ -1,7 +1,7 @@
 """Device memory of the cache, laid out for the groups the model's layers form.
 
 `CacheLayout` reads a model's schedule: runs whose mixers keep paged keys/values with the
-same (kv heads, head size, window, parts) form a group; each writing run gets a plane of its own in
+same (kv heads, head size, window, parts, kept first positions) form a group; each writing run gets a plane of its own in
 the group's pool, a run with `cache_of` shares the plane of the run it names (it may look back
 over another window: the plane then keeps what the widest of its readers needs).  Runs whose
 mixers (or blocks) keep a fixed-size state get a state array [max_requests, ...] indexed by slot
@@ -38,12 +38,15 @@ class CacheLayout:
         self.needs = model.cache_needs()
         self.schedule = model.schedule
         self.group_keys: List[tuple] = []
+        self.group_keep_first: List[int] = []
         self.group_planes: List[int] = []
         self.run_group: List[Optional[int]] = []
         self.run_plane: List[Optional[int]] = []
         self.run_state: List[Optional[int]] = []
         self.state_needs = []
         # the window a writing run's plane must keep: the widest of the runs that read it (0: everything)
+        first = {k: need.paged.keep_first for k, (run, need) in enumerate(zip(self.schedule, self.needs))
+                 if run.cache_of is None and need.paged is not None}
         keep = {k: [need.paged.window] for k, (run, need) in enumerate(zip(self.schedule, self.needs))
                 if run.cache_of is None and need.paged is not None}
         for k, (run, need) in enumerate(zip(self.schedule, self.needs)):
@@ -55,6 +58,7 @@ class CacheLayout:
                     raise ValueError(f"run {k} cannot read the cache of run {j}: their needs differ")
                 if a is not None:
                     keep[j].append(a.window)
+                    first[j] = max(first[j], a.keep_first)
         for k, (run, need) in enumerate(zip(self.schedule, self.needs)):
             if run.cache_of is not None:
                 j = run.cache_of
@@ -63,10 +67,12 @@ class CacheLayout:
             elif need.paged is not None:
                 window = 0 if min(keep[k]) <= 0 else max(keep[k])
                 key = (need.paged.n_kv_heads, need.paged.head_dim, window, need.paged.parts)
-                if key not in self.group_keys:
+                kept = first[k] if window else 0
+                if (key, kept) not in zip(self.group_keys, self.group_keep_first):
                     self.group_keys.append(key)
+                    self.group_keep_first.append(kept)
                     self.group_planes.append(0)
-                g = self.group_keys.index(key)
+                g = list(zip(self.group_keys, self.group_keep_first)).index((key, kept))
                 self.run_group.append(g)
                 self.run_plane.append(self.group_planes[g])
                 self.group_planes[g] += 1
@@ -99,7 +105,8 @@ class CacheStorage:
             num_pages = (int(max_tokens) + self.page_size - 1) // self.page_size
         pages = list(num_pages) if isinstance(num_pages, (list, tuple)) else [int(num_pages)] * n_groups
         self.table_width = (max_model_len + self.page_size - 1) // self.page_size
-        specs = [host.module().GroupSpec(self.page_size, key[2], pages[g], self.table_width)
+        specs = [host.module().GroupSpec(self.page_size, key[2], pages[g], self.table_width,
+                                         self.layout.group_keep_first[g])
                  for g, key in enumerate(self.layout.group_keys)]
         if not specs:   # a model without paged layers still needs slots and lengths: pages without memory
             specs = [host.module().GroupSpec(self.page_size, 0, int(max_requests) * self.table_width, self.table_width)]

@@ -93,3 +93,5 @@ def _ensure_builtin():
         from ..models import zavesun  # noqa: F401
     if "Pererax" not in _REGISTRY:
         from ..models import pererax  # noqa: F401
+    if "Tikunex" not in _REGISTRY:
+        from ..models import tikunex  # noqa: F401

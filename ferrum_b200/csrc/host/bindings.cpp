@@ -36,19 +36,22 @@ PYBIND11_MODULE(_host, m) {
   });
 
   py::class_<GroupSpec>(m, "GroupSpec")
-      .def(py::init([](int page_size, int window, int num_pages, int table_width) {
+      .def(py::init([](int page_size, int window, int num_pages, int table_width, int keep_first) {
              GroupSpec g;
              g.page_size = page_size;
              g.window = window;
              g.num_pages = num_pages;
              g.table_width = table_width;
+             g.keep_first = keep_first;
              return g;
            }),
-           py::arg("page_size"), py::arg("window"), py::arg("num_pages"), py::arg("table_width"))
+           py::arg("page_size"), py::arg("window"), py::arg("num_pages"), py::arg("table_width"),
+           py::arg("keep_first") = 0)
       .def_readonly("page_size", &GroupSpec::page_size)
       .def_readonly("window", &GroupSpec::window)
       .def_readonly("num_pages", &GroupSpec::num_pages)
-      .def_readonly("table_width", &GroupSpec::table_width);
+      .def_readonly("table_width", &GroupSpec::table_width)
+      .def_readonly("keep_first", &GroupSpec::keep_first);
 
   py::class_<CacheManager>(m, "CacheManager")
       .def(py::init<std::vector<GroupSpec>, int>(), py::arg("groups"), py::arg("max_requests"))

@@ -8,7 +8,7 @@ CacheManager::CacheManager(std::vector<GroupSpec> groups, int max_requests)
     : groups_(std::move(groups)), max_requests_(max_requests) {
   if (max_requests_ <= 0) throw CacheError("cache: max_requests must be positive");
   for (auto& g : groups_) {
-    if (g.page_size <= 0 || g.num_pages <= 0 || g.table_width <= 0 || g.window < 0)
+    if (g.page_size <= 0 || g.num_pages <= 0 || g.table_width <= 0 || g.window < 0 || g.keep_first < 0)
       throw CacheError("cache: a group dimension is zero or negative");
   }
   reqs_.resize(max_requests_);
@@ -68,6 +68,11 @@ int CacheManager::first_needed_page(int g, int pos0) const {
   return lo / s.page_size;
 }
 
+int CacheManager::kept_pages(int g) const {
+  const GroupSpec& s = groups_[g];
+  return (s.keep_first + s.page_size - 1) / s.page_size;
+}
+
 std::vector<int> CacheManager::pages_missing(int slot, int new_len) const {
   check_slot(slot);
   const Req& r = reqs_[slot];
@@ -124,7 +129,7 @@ void CacheManager::commit(int slot, int new_len) {
   // pages that no later query reaches: the next query stands at new_len
   for (size_t g = 0; g < groups_.size(); ++g) {
     const int keep_from = first_needed_page((int)g, new_len);
-    for (int lp = 0; lp < keep_from; ++lp) {
+    for (int lp = kept_pages((int)g); lp < keep_from; ++lp) {
       int32_t& p = r.tables[g][lp];
       if (p >= 0) {
         in_use_[g][p] = 0;

@@ -5,7 +5,8 @@
 // `page_size` positions.  Layers with the same needs form a group; every group has its own
 // pool of pages and every request has one block table per group (logical page -> page id,
 // -1 where it holds none).  A group with a window gives pages back as soon as no later
-// query can reach them.  Beside the pages, every request owns one slot id, which indexes
+// query can reach them; the pages of a sequence's first `keep_first` positions stay, where its
+// layers see those positions from everywhere.  Beside the pages, every request owns one slot id, which indexes
 // arrays of fixed-size per-request state.
 //
 // The manager owns integers only; the device memory the page ids index belongs to the caller.
@@ -25,6 +26,7 @@ struct GroupSpec {
   int window = 0;       // 0: every key is kept; w > 0: a query at p reads keys in (p - w, p]
   int num_pages = 0;
   int table_width = 0;  // logical pages a request may address
+  int keep_first = 0;   // with a window: the positions 0 .. keep_first - 1 are seen by every later query too
 };
 
 class CacheManager {
@@ -78,6 +80,8 @@ class CacheManager {
   void check_slot(int slot) const;
   // first logical page a step starting at position pos0 still needs in group g
   int first_needed_page(int g, int pos0) const;
+  // pages at the front of a sequence that group g never gives back before the request ends
+  int kept_pages(int g) const;
 
   std::vector<GroupSpec> groups_;
   int max_requests_;

@@ -24,7 +24,10 @@
 // `window` > 0 keeps keys in (pos-window, pos]; with `chunked` the same number is the length of a
 // chunk instead: positions are cut into chunks of `window` from position 0 and a query sees the
 // keys of its own chunk up to itself.  `softcap` c > 0 bends the scaled score to c * tanh(score / c)
-// (before any distance penalty).  `sink`: a key of score 0 without a value joins every row's softmax,
+// (before any distance penalty).  `keep_first` > 0: beside its window a query sees the sequence's first
+// keep_first keys (up to itself); the walk goes over those of them that lie before the window (or before the
+// first key that any row of a token tile sees), then over the window; with splits they are splits of their own,
+// numbered before the window's.  `sink`: a key of score 0 without a value joins every row's softmax,
 // weight_j = exp(s_j) / (exp(0) + sum exp(s)); it enters once, where a row's (maximum, sum, values)
 // are final: in the walking kernels' last step, or in the fold of the splits.
 #include "common.cuh"
@@ -121,6 +124,11 @@ __device__ __forceinline__ int ag_first_key(int pos, int window, int chunked) {
   return chunked ? (pos / window) * window : max(0, pos - window + 1);
 }
 
+// Kept first keys that lie before `lo`, which are walked before the keys from `lo` on.
+__device__ __forceinline__ int ag_kept(int lo, int keep_first) { return min(keep_first, lo); }
+// Splits that kept keys may take (0 without any): slot s < this number holds kept keys s * AG_SPLIT .. .
+__host__ __device__ __forceinline__ int ag_kept_splits(int keep_first) { return (keep_first + AG_SPLIT - 1) / AG_SPLIT; }
+
 // part: null (the CTA covers the row's whole key range and writes `out`), or the partials
 // [token][head][split slot][D + 2] of the split that blockIdx.y names.
 // The tile after the one being worked on is on its way meanwhile: float32 rows that are 16-byte
@@ -134,7 +142,7 @@ attention_generic_kernel(const T* __restrict__ q, int ldq, T* __restrict__ out, 
                          long long page_stride, int page_size, int Hq, int Hkv, int D, float scale, int window,
                          int* __restrict__ err, float* __restrict__ part, int split_slots, int vec,
                          const float* __restrict__ bias1, const float* __restrict__ bias2, int out_f32, int chunked,
-                         float softcap, int sink) {
+                         float softcap, int sink, int keep_first, float out_scale) {
   using Tile = AgTile<DI>;
   constexpr int TK = Tile::TK, DP = Tile::DP, KS = Tile::KS;
   extern __shared__ __align__(16) float ag_smem[];
@@ -153,23 +161,33 @@ attention_generic_kernel(const T* __restrict__ q, int ldq, T* __restrict__ out, 
   const int nh = min(AG_HEADS, G - chunk * AG_HEADS);
   const int pos = positions[t];
   const int lo = ag_first_key(pos, window, chunked);
-  int k_begin = lo, k_end = pos + 1;
+  int k_begin = lo, k_end = pos + 1, kept = ag_kept(lo, keep_first);      // keys 0 .. kept - 1, then k_begin .. k_end - 1
   if (part != nullptr) {
-    const int s = lo / AG_SPLIT + blockIdx.y;
-    if (s * AG_SPLIT > pos) return;            // this row has fewer splits
-    k_begin = max(lo, s * AG_SPLIT);
-    k_end = min(pos + 1, (s + 1) * AG_SPLIT);
+    const int kept_splits = ag_kept_splits(keep_first);
+    if ((int)blockIdx.y < kept_splits) {
+      k_begin = blockIdx.y * AG_SPLIT;
+      k_end = min(kept, k_begin + AG_SPLIT);
+      if (k_begin >= k_end) return;            // these kept keys are in the row's window
+    } else {
+      const int s = lo / AG_SPLIT + blockIdx.y - kept_splits;
+      if (s * AG_SPLIT > pos) return;          // this row has fewer splits
+      k_begin = max(lo, s * AG_SPLIT);
+      k_end = min(pos + 1, (s + 1) * AG_SPLIT);
+    }
+    kept = 0;
   }
+  // the key at place n of the walk
+  auto key_at = [&](int n) { return n < kept ? n : k_begin + n - kept; };
   const int* bt = block_table + (size_t)req_of_token[t] * table_width;
   const size_t v_off = (size_t)Hkv * page_size * D;
   const bool vec_ok = vec != 0;
   const bool async_rows = vec_ok && sizeof(T) == 4;
-  const int n_tiles = (k_end - k_begin + TK - 1) / TK;
+  const int n_tiles = (kept + k_end - k_begin + TK - 1) / TK;
 
   // where the rows of tile n lie (threads 0 .. TK-1)
   auto find_rows = [&](int n) {
     if (threadIdx.x < TK) {
-      const int key = k_begin + n * TK + threadIdx.x;
+      const int key = key_at(n * TK + threadIdx.x);
       long long off = -1;
       if (key < k_end) {
         const int lp = key / page_size;
@@ -291,7 +309,7 @@ attention_generic_kernel(const T* __restrict__ q, int ldq, T* __restrict__ out, 
           dot = fmaf(a.z, k4.z, dot);
           dot = fmaf(a.w, k4.w, dot);
         }
-        s = ag_score(dot, scale, softcap) - ag_distance_penalty(bias1, bias2, h0 + warp, pos - (k_begin + n * TK + lane));
+        s = ag_score(dot, scale, softcap) - ag_distance_penalty(bias1, bias2, h0 + warp, pos - key_at(n * TK + lane));
       }
       const float m_new = fmaxf(m, warp_max(s));
       float corr = 1.f, pj = 0.f;
@@ -335,7 +353,7 @@ attention_generic_kernel(const T* __restrict__ q, int ldq, T* __restrict__ out, 
 #pragma unroll
     for (int i = 0; i < DI; ++i) {
       const int d = lane + 32 * i;
-      if (d < D) ag_store<T>(out, (size_t)t * ldo + (size_t)h * D + d, l > 0.f ? acc[i] * f / l : 0.f, out_f32);
+      if (d < D) ag_store<T>(out, (size_t)t * ldo + (size_t)h * D + d, l > 0.f ? acc[i] * f / l * out_scale : 0.f, out_f32);
     }
   } else {
     float* p = part + (((size_t)t * Hq + h) * split_slots + blockIdx.y) * (D + 2);
@@ -385,7 +403,8 @@ attention_generic_tokens_kernel(const T* __restrict__ q, int ldq, T* __restrict_
                                 const int* __restrict__ block_table, int table_width, const T* __restrict__ kv_plane,
                                 long long page_stride, int page_size, int Hq, int Hkv, int D, float scale, int window,
                                 int* __restrict__ err, int vec, const float* __restrict__ bias1,
-                                const float* __restrict__ bias2, int out_f32, int chunked, float softcap, int sink) {
+                                const float* __restrict__ bias2, int out_f32, int chunked, float softcap, int sink, int keep_first,
+                                float out_scale) {
   using Tile = AgTile<DI>;
   using TT = AgTokenTile<DI>;
   constexpr int TK = Tile::TK, DP = Tile::DP, KS = Tile::KS;
@@ -444,11 +463,13 @@ attention_generic_tokens_kernel(const T* __restrict__ q, int ldq, T* __restrict_
   const size_t v_off = (size_t)Hkv * page_size * D;
   const bool vec_ok = vec != 0;
   const bool async_rows = vec_ok && sizeof(T) == 4;
-  const int n_tiles = (k_end - k_begin + TK - 1) / TK;
+  const int kept = ag_kept(k_begin, keep_first);      // keys 0 .. kept - 1, then k_begin .. k_end - 1
+  auto key_at = [&](int n) { return n < kept ? n : k_begin + n - kept; };
+  const int n_tiles = (kept + k_end - k_begin + TK - 1) / TK;
 
   auto find_rows = [&](int n) {
     if (threadIdx.x < TK) {
-      const int key = k_begin + n * TK + threadIdx.x;
+      const int key = key_at(n * TK + threadIdx.x);
       long long off = -1;
       if (key < k_end) {
         const int lp = key / page_size;
@@ -517,7 +538,7 @@ attention_generic_tokens_kernel(const T* __restrict__ q, int ldq, T* __restrict_
     if (warp < nh) {
       const float* const kb = sm_k + b * TK * KS;
       const float* const vb = sm_v + b * TK * DP;
-      const int key = k_begin + n * TK + lane;
+      const int key = key_at(n * TK + lane);
       // ---- lane j: the scores of key j for this warp's head and the chunk's tokens
       float sc[AG_TH];
 #pragma unroll
@@ -541,7 +562,7 @@ attention_generic_tokens_kernel(const T* __restrict__ q, int ldq, T* __restrict_
       __syncwarp();                             // the weights of the tile before have been read
 #pragma unroll
       for (int i = 0; i < AG_TH; ++i) {
-        const bool seen = have && key <= pos[i] && key >= lo[i];
+        const bool seen = have && key <= pos[i] && (key >= lo[i] || key < keep_first);
         const float sv = seen ? ag_score(sc[i], scale, softcap) - ag_distance_penalty(bias1, bias2, h0 + warp, pos[i] - key) : -INFINITY;
         const float m_new = fmaxf(m[i], warp_max(sv));
         float cr = 1.f, pj = 0.f;
@@ -594,7 +615,7 @@ attention_generic_tokens_kernel(const T* __restrict__ q, int ldq, T* __restrict_
 #pragma unroll
     for (int e = 0; e < DI; ++e) {
       const int d = lane + 32 * e;
-      if (d < D) ag_store<T>(out, (size_t)(t0 + i0 + i) * ldo + (size_t)h * D + d, li > 0.f ? acc[i][e] * f / li : 0.f, out_f32);
+      if (d < D) ag_store<T>(out, (size_t)(t0 + i0 + i) * ldo + (size_t)h * D + d, li > 0.f ? acc[i][e] * f / li * out_scale : 0.f, out_f32);
     }
   }
 }
@@ -603,11 +624,13 @@ attention_generic_tokens_kernel(const T* __restrict__ q, int ldq, T* __restrict_
 template <typename T>
 __global__ void __launch_bounds__(32)
 attention_generic_combine_kernel(T* __restrict__ out, int ldo, const float* __restrict__ part, const int* __restrict__ positions,
-                                 int Hq, int D, int window, int split_slots, int out_f32, int chunked, int sink) {
+                                 int Hq, int D, int window, int split_slots, int out_f32, int chunked, int sink, int keep_first,
+                                 float out_scale) {
   const int t = blockIdx.x, h = blockIdx.y, lane = threadIdx.x;
   const int pos = positions[t];
   const int lo = ag_first_key(pos, window, chunked);
-  const int n = pos / AG_SPLIT - lo / AG_SPLIT + 1;
+  const int kept = ag_kept(lo, keep_first), kept_splits = ag_kept_splits(keep_first);
+  const int n = kept_splits + pos / AG_SPLIT - lo / AG_SPLIT + 1;
   const float* base = part + ((size_t)t * Hq + h) * split_slots * (D + 2);
   float M = -INFINITY, L = 0.f, O[AG_DI];
 #pragma unroll
@@ -617,7 +640,7 @@ attention_generic_combine_kernel(T* __restrict__ out, int ldo, const float* __re
     float mb[4], lb[4], ob[4][AG_DI];
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      const bool have = s0 + j < total;
+      const bool have = s0 + j < total && (s0 + j >= kept_splits || (s0 + j) * AG_SPLIT < kept);
       const float* p = base + (size_t)(have ? s0 + j : 0) * (D + 2);
       mb[j] = have ? p[0] : -INFINITY;
       lb[j] = have ? p[1] : 0.f;
@@ -644,7 +667,7 @@ attention_generic_combine_kernel(T* __restrict__ out, int ldo, const float* __re
 #pragma unroll
   for (int i = 0; i < AG_DI; ++i) {
     const int d = lane + 32 * i;
-    if (d < D) ag_store<T>(out, (size_t)t * ldo + (size_t)h * D + d, L > 0.f ? O[i] * f / L : 0.f, out_f32);
+    if (d < D) ag_store<T>(out, (size_t)t * ldo + (size_t)h * D + d, L > 0.f ? O[i] * f / L * out_scale : 0.f, out_f32);
   }
 }
 
@@ -658,7 +681,7 @@ FERRUM_API int ferrum_attention_generic_split() { return AG_SPLIT; }
 // and a second launch folds the partials into `out`.
 // bias1, bias2 (float32 per query head on the device, or null): the distance penalty above.  out_f32: the
 // output rows are float32 whatever the cache's type.  chunked: `window` is a chunk length (see the top).
-// softcap, sink: see the top.
+// softcap, sink, keep_first: see the top; out_scale multiplies every output element (1: none).
 // q_start (n_reqs + 1 entries on the device; may be null): with it and without `part`, tokens of a
 // request that follow each other in the batch share their key tiles (the kernel for prompt portions).
 FERRUM_API int ferrum_attention_generic(const void* q, int ldq, void* out, int ldo, int dtype, int n_tokens,
@@ -666,14 +689,15 @@ FERRUM_API int ferrum_attention_generic(const void* q, int ldq, void* out, int l
                                         int table_width, const void* kv_plane, long long page_stride, int page_size,
                                         int Hq, int Hkv, int D, float scale, int window, int* err_flag, float* part,
                                         int split_slots, const int* q_start, int n_reqs, const float* bias1,
-                                        const float* bias2, int out_f32, int chunked, float softcap, int sink,
-                                        cudaStream_t stream) {
+                                        const float* bias2, int out_f32, int chunked, float softcap, int sink, int keep_first,
+                                        float out_scale, cudaStream_t stream) {
   FERRUM_CHECK_ARG(n_tokens >= 0 && Hq > 0 && Hkv > 0 && Hq % Hkv == 0, "attention: bad head counts Hq=%d Hkv=%d", Hq, Hkv);
   FERRUM_CHECK_ARG(D > 0 && D <= AG_MAX_D, "attention: head size %d is outside (0, %d]", D, AG_MAX_D);
-  FERRUM_CHECK_ARG(page_size > 0 && table_width > 0 && window >= 0, "attention: bad cache arguments");
+  FERRUM_CHECK_ARG(page_size > 0 && table_width > 0 && window >= 0 && keep_first >= 0, "attention: bad cache arguments");
   FERRUM_CHECK_ARG(ldq >= Hq * D && ldo >= Hq * D, "attention: a row stride is shorter than Hq*D");
   FERRUM_CHECK_ARG(part == nullptr || (split_slots > 0 && split_slots <= 65535), "attention: bad number of split slots %d", split_slots);
   if (n_tokens == 0) return 0;
+  if (window == 0) keep_first = 0;             // every earlier key is seen anyway
   const int G = Hq / Hkv;
   const long long rows = (long long)n_tokens * Hkv * ((G + AG_HEADS - 1) / AG_HEADS);
   FERRUM_CHECK_ARG(rows < (1LL << 31), "attention: too many rows");
@@ -696,7 +720,7 @@ FERRUM_API int ferrum_attention_generic(const void* q, int ldq, void* out, int l
     }                                                                                                                   \
     attention_generic_tokens_kernel<T, DI_><<<(unsigned)ctas, AG_TWARPS * 32, AgTokenTile<DI_>::SMEM_BYTES, stream>>>(   \
       (const T*)q, ldq, (T*)out, ldo, positions, q_start, n_reqs, block_table, table_width, (const T*)kv_plane,         \
-      page_stride, page_size, Hq, Hkv, D, scale, window, err_flag, vec, bias1, bias2, out_f32, chunked, softcap, sink);                                        \
+      page_stride, page_size, Hq, Hkv, D, scale, window, err_flag, vec, bias1, bias2, out_f32, chunked, softcap, sink, keep_first, out_scale);                \
   })
     if (D <= 32) AG_LAUNCH_TOKENS(1);
     else if (D <= 64) AG_LAUNCH_TOKENS(2);
@@ -719,7 +743,7 @@ FERRUM_API int ferrum_attention_generic(const void* q, int ldq, void* out, int l
     }                                                                                                                   \
     attention_generic_kernel<T, DI_><<<grid, AG_WARPS * 32, AgTile<DI_>::SMEM_BYTES, stream>>>(                        \
       (const T*)q, ldq, (T*)out, ldo, positions, req_of_token, block_table, table_width, (const T*)kv_plane, page_stride, \
-      page_size, Hq, Hkv, D, scale, window, err_flag, part, split_slots, vec, bias1, bias2, out_f32, chunked, softcap, sink);                                  \
+      page_size, Hq, Hkv, D, scale, window, err_flag, part, split_slots, vec, bias1, bias2, out_f32, chunked, softcap, sink, keep_first, out_scale);          \
   })
   if (D <= 32) AG_LAUNCH(1);
   else if (D <= 64) AG_LAUNCH(2);
@@ -731,7 +755,7 @@ FERRUM_API int ferrum_attention_generic(const void* q, int ldq, void* out, int l
     const dim3 cgrid(n_tokens, Hq);
     FERRUM_CHECK_ARG(cgrid.y <= 65535, "attention: too many heads");
     FERRUM_DISPATCH_DTYPE(dtype, T, (attention_generic_combine_kernel<T><<<cgrid, 32, 0, stream>>>(
-        (T*)out, ldo, part, positions, Hq, D, window, split_slots, out_f32, chunked, sink)));
+        (T*)out, ldo, part, positions, Hq, D, window, split_slots, out_f32, chunked, sink, keep_first, out_scale)));
     FERRUM_CHECK_LAUNCH("attention_generic_combine");
   }
   return 0;

@@ -18,7 +18,7 @@
 //
 // attention_finish: reads the attention's float32 output [T, Hq, Dp]; turns each head back by the
 // query's position (the inverse of the value rotation), multiplies by a sigmoid gate whose logits lie
-// in the product's row, and writes [T, Hq, Dv] in the compute type for the output projection.
+// in the product's row, by a constant, and writes [T, Hq, Dv] in the compute type for the output projection.
 //
 // One warp per (token, head).  Every step of a head is float32; the only rounding is the store.
 #include "common.cuh"
@@ -145,7 +145,7 @@ template <typename T>
 __global__ void __launch_bounds__(AP_WARPS * 32)
 attention_finish_kernel(const float* __restrict__ o, int ldo, int n_tokens, const int* __restrict__ positions,
                         const float* __restrict__ cs_v, int v_pairing, int n_pos_v, const float* __restrict__ gate,
-                        int ldg, T* __restrict__ out, int ldout, int Hq, int Dv, int Dp, int* __restrict__ err) {
+                        int ldg, T* __restrict__ out, int ldout, int Hq, int Dv, int Dp, int* __restrict__ err, float out_scale) {
   pdl_launch();      // the product that follows may fetch its weights meanwhile
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long item = (long long)blockIdx.x * AP_WARPS + warp;
@@ -170,14 +170,14 @@ attention_finish_kernel(const float* __restrict__ o, int ldo, int n_tokens, cons
         ra *= 1.f / (1.f + expf(-g[a]));
         rb *= 1.f / (1.f + expf(-g[b]));
       }
-      dst[a] = from_f32<T>(ra);
-      dst[b] = from_f32<T>(rb);
+      dst[a] = from_f32<T>(ra * out_scale);
+      dst[b] = from_f32<T>(rb * out_scale);
     }
   } else {
     for (int d = lane; d < Dv; d += 32) {
       float r = src[d];
       if (g != nullptr) r *= 1.f / (1.f + expf(-g[d]));
-      dst[d] = from_f32<T>(r);
+      dst[d] = from_f32<T>(r * out_scale);
     }
   }
 }
@@ -215,14 +215,14 @@ FERRUM_API int ferrum_qkv_shape(const float* proj, int ldp, int n_tokens, const 
 
 FERRUM_API int ferrum_attention_finish(const float* o, int ldo, int n_tokens, const int* positions, const float* cs_v,
                                        int v_pairing, int n_pos_v, const float* gate, int ldg, void* out, int ldout,
-                                       int dtype, int Hq, int Dv, int Dp, int* err, cudaStream_t stream) {
+                                       int dtype, int Hq, int Dv, int Dp, int* err, float out_scale, cudaStream_t stream) {
   FERRUM_CHECK_ARG(Hq > 0 && Dv > 0 && Dp >= Dv, "attention_finish: bad head sizes Dv=%d Dp=%d", Dv, Dp);
   FERRUM_CHECK_ARG(cs_v == nullptr || Dv % 2 == 0, "attention_finish: a rotated value needs an even size");
   if (n_tokens == 0) return 0;
   const long long blocks = ((long long)n_tokens * Hq + AP_WARPS - 1) / AP_WARPS;
   FERRUM_CHECK_ARG(blocks < (1LL << 31), "attention_finish: too many rows");
   FERRUM_DISPATCH_DTYPE(dtype, T, (attention_finish_kernel<T><<<(unsigned)blocks, AP_WARPS * 32, 0, stream>>>(
-      o, ldo, n_tokens, positions, cs_v, v_pairing, n_pos_v, gate, ldg, (T*)out, ldout, Hq, Dv, Dp, err)));
+      o, ldo, n_tokens, positions, cs_v, v_pairing, n_pos_v, gate, ldg, (T*)out, ldout, Hq, Dv, Dp, err, out_scale)));
   FERRUM_CHECK_LAUNCH("attention_finish");
   return 0;
 }

@@ -37,6 +37,41 @@ FERRUM_API int ferrum_embedding(const void* table, int dtype, const int* ids, fl
   return 0;
 }
 
+// The embedded row through an RMS norm: out[t] = rms(table[ids[t]]) * w, float32; the result may also be left in the
+// compute type (`copy`, rows of ldc elements: what a later product reads again).
+template <typename T>
+__global__ void __launch_bounds__(256)
+embedding_norm_kernel(const T* __restrict__ table, const int* __restrict__ ids, const float* __restrict__ w, float eps,
+                      float* __restrict__ out, T* __restrict__ copy, int ldc, int E, int V, int* __restrict__ err) {
+  __shared__ float red[32];
+  const int t = blockIdx.x;
+  const int id = ids[t];
+  const bool ok = id >= 0 && id < V;
+  if (!ok && threadIdx.x == 0) atomicExch(err, 1);
+  const T* row = table + (size_t)(ok ? id : 0) * E;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < E; i += 256) {
+    const float v = ok ? to_f32<T>(row[i]) : 0.f;
+    ss = fmaf(v, v, ss);
+  }
+  ss = block_sum(ss, red);
+  const float inv = 1.0f / sqrtf(ss / (float)E + eps);
+  for (int i = threadIdx.x; i < E; i += 256) {
+    const float v = ok ? to_f32<T>(row[i]) * inv * w[i] : 0.f;
+    out[(size_t)t * E + i] = v;
+    if (copy != nullptr) copy[(size_t)t * ldc + i] = from_f32<T>(v);
+  }
+}
+
+FERRUM_API int ferrum_embedding_norm(const void* table, int dtype, const int* ids, const float* w, float eps, float* out, void* copy,
+                                     int ldc, int n_tokens, int E, int V, int* err_flag, cudaStream_t stream) {
+  FERRUM_CHECK_ARG(n_tokens >= 0 && E > 0 && V > 0 && (copy == nullptr || ldc >= E), "embedding_norm: bad sizes T=%d E=%d V=%d", n_tokens, E, V);
+  if (n_tokens == 0) return 0;
+  FERRUM_DISPATCH_DTYPE(dtype, T, (embedding_norm_kernel<T><<<n_tokens, 256, 0, stream>>>((const T*)table, ids, w, eps, out, (T*)copy, ldc, E, V, err_flag)));
+  FERRUM_CHECK_LAUNCH("embedding_norm");
+  return 0;
+}
+
 // ---------------------------------------------------------------- RMSNorm
 // out[r, i] = x[src(r), i] * rsqrt(mean(x^2) + eps) * w[i]; src(r) = rows ? rows[r] : r.
 // One block per row, the same reduction tree for every row.

@@ -1,7 +1,7 @@
 // A routed feed-forward: every token goes through `top` of `n_exp` small gated feed-forwards.
 //
-// moe_route   one warp per token: scores from the router's float32 logits (sigmoid of each, or a
-//             softmax over all), the `top` largest (ties: the lower index), optionally renormalised to
+// moe_route   one warp per token: scores from the router's float32 logits, to which a bias may be added
+//             (sigmoid of each, a softmax over all, or a softmax over the chosen logits only), the `top` largest (ties: the lower index), optionally renormalised to
 //             sum 1; the token takes a place in each chosen expert's group (an atomic counter per expert).
 //             A correction vector may be added to the scores for the choice alone (the weights stay the
 //             plain scores), the weights may be multiplied by a constant, and the last router outputs may
@@ -26,13 +26,14 @@
 
 constexpr int MOE_MAX_EXPERTS = 256;
 constexpr int MOE_MAX_TOP = 8;
+enum MoeScores : int { MOE_SIGMOID = 0, MOE_SOFTMAX = 1, MOE_CHOSEN_SOFTMAX = 2 };
 
 // ------------------------------------------------------------------ routing
 // logits [T][ldz] float32.  expert_of, rank_of [T*top] int32, weight_of [T*top] float32, counts [n_exp] (zero on entry).
 __global__ void __launch_bounds__(128)
-moe_route_kernel(const float* __restrict__ logits, int ldz, int n_tokens, int n_exp, int top, int softmax_scores, int renormalize,
+moe_route_kernel(const float* __restrict__ logits, int ldz, int n_tokens, int n_exp, int top, int score_kind, int renormalize,
                  int* __restrict__ expert_of, int* __restrict__ rank_of, float* __restrict__ weight_of, int* __restrict__ counts,
-                 const float* __restrict__ correction, float weight_scale, int n_real) {
+                 const float* __restrict__ correction, float weight_scale, int n_real, const float* __restrict__ bias) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * 4 + warp;
   if (t >= n_tokens) return;
@@ -42,10 +43,10 @@ moe_route_kernel(const float* __restrict__ logits, int ldz, int n_tokens, int n_
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
     const int e = lane + 32 * i;
-    s[i] = e < n_exp ? logits[(size_t)t * ldz + e] : -INFINITY;
+    s[i] = e < n_exp ? logits[(size_t)t * ldz + e] + (bias != nullptr ? bias[e] : 0.f) : -INFINITY;
     mx = fmaxf(mx, s[i]);
   }
-  if (softmax_scores) {
+  if (score_kind == MOE_SOFTMAX) {
     mx = warp_max(mx);
     float sum = 0.f;
 #pragma unroll
@@ -57,7 +58,7 @@ moe_route_kernel(const float* __restrict__ logits, int ldz, int n_tokens, int n_
 #pragma unroll
     for (int i = 0; i < PER; ++i)
       if (lane + 32 * i < n_exp) s[i] /= sum;
-  } else {
+  } else if (score_kind == MOE_SIGMOID) {
 #pragma unroll
     for (int i = 0; i < PER; ++i)
       if (lane + 32 * i < n_exp) s[i] = 1.f / (1.f + expf(-s[i]));
@@ -100,6 +101,15 @@ moe_route_kernel(const float* __restrict__ logits, int ldz, int n_tokens, int n_
 #pragma unroll
     for (int i = 0; i < PER; ++i)
       if (lane + 32 * i == best_e) pick[i] = -INFINITY;
+  }
+  if (score_kind == MOE_CHOSEN_SOFTMAX) {   // (so far the scores are the logits, the largest first)
+    float sum = 0.f;
+    const float top_logit = chosen_w[0];
+    for (int j = 0; j < top; ++j) {
+      chosen_w[j] = expf(chosen_w[j] - top_logit);
+      sum += chosen_w[j];
+    }
+    for (int j = 0; j < top; ++j) chosen_w[j] /= sum;
   }
   if (lane == 0) {
     for (int j = 0; j < top; ++j) {
@@ -562,12 +572,13 @@ int run(const void* A, int lda, const void* W, int w_rows, int K, int N, int n_e
 // y[t][:] = sum over the token's choices, in their order, of rows[row_of[t*top + j]][:] (float32), each times
 // weight_of[t*top + j] when that is given; for consumers that want a plain buffer.  A choice without a row
 // (row_of < 0: an identity expert) stands for the token's own input row x[t][:]; `add` (float32 rows, may be null:
-// a unit that every token runs through) joins the sum last.
+// a unit that every token runs through) joins the sum last.  `accumulate`: y (a residual stream) gains the sum instead of
+// being overwritten; yc (the type of x; may be null) receives the new y.
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ rows, int ld, const int* __restrict__ row_of, const float* __restrict__ weight_of,
                    int top, int E, float* __restrict__ y, const T* __restrict__ x, int ldx, const float* __restrict__ add,
-                   int ld_add) {
+                   int ld_add, int accumulate, T* __restrict__ yc, int ldyc) {
   const int t = blockIdx.x;
   for (int i = threadIdx.x; i < E; i += 256) {
     float s = 0.f;
@@ -577,7 +588,9 @@ moe_combine_kernel(const float* __restrict__ rows, int ld, const int* __restrict
       s += weight_of != nullptr ? v * weight_of[(size_t)t * top + j] : v;
     }
     if (add != nullptr) s += add[(size_t)t * ld_add + i];
+    if (accumulate) s = y[(size_t)t * E + i] + s;
     y[(size_t)t * E + i] = s;
+    if (yc != nullptr) yc[(size_t)t * ldyc + i] = from_f32<T>(s);
   }
 }
 
@@ -592,10 +605,12 @@ FERRUM_API int ferrum_moe_max_experts() { return MOE_MAX_EXPERTS; }
 FERRUM_API int ferrum_moe_max_top() { return MOE_MAX_TOP; }
 
 // Routing and gathering of one step.  counts: n_exp ints (zeroed here).
-FERRUM_API int ferrum_moe_route(const float* logits, int ldz, int n_tokens, int n_exp, int top, int softmax_scores,
+FERRUM_API int ferrum_moe_route(const float* logits, int ldz, int n_tokens, int n_exp, int top, int score_kind,
                                 int renormalize, const void* x, int ldx, int E, int dtype, int scale_input, int* expert_of,
                                 int* rank_of, float* weight_of, int* counts, void* xg, int* row_of, const float* correction,
-                                float weight_scale, int n_identity, cudaStream_t stream) {
+                                float weight_scale, int n_identity, const float* bias, cudaStream_t stream) {
+  FERRUM_CHECK_ARG(score_kind >= MOE_SIGMOID && score_kind <= MOE_CHOSEN_SOFTMAX && (score_kind != MOE_CHOSEN_SOFTMAX || correction == nullptr),
+                   "moe_route: a softmax over the chosen logits takes no correction");
   FERRUM_CHECK_ARG(n_exp > 0 && n_exp <= MOE_MAX_EXPERTS && top > 0 && top <= MOE_MAX_TOP && top <= n_exp,
                    "moe_route: %d experts, %d per token are outside the kernel's limits (%d, %d)", n_exp, top, MOE_MAX_EXPERTS, MOE_MAX_TOP);
   FERRUM_CHECK_ARG(n_identity >= 0 && n_identity < n_exp, "moe_route: %d identity experts among %d router outputs", n_identity, n_exp);
@@ -605,8 +620,8 @@ FERRUM_API int ferrum_moe_route(const float* logits, int ldz, int n_tokens, int 
   if (n_tokens == 0) return 0;
   cudaError_t e = cudaMemsetAsync(counts, 0, sizeof(int) * n_real, stream);
   FERRUM_CHECK_ARG(e == cudaSuccess, "moe_route: cannot clear the counters: %s", cudaGetErrorString(e));
-  moe_route_kernel<<<(n_tokens + 3) / 4, 128, 0, stream>>>(logits, ldz, n_tokens, n_exp, top, softmax_scores, renormalize,
-                                                           expert_of, rank_of, weight_of, counts, correction, weight_scale, n_real);
+  moe_route_kernel<<<(n_tokens + 3) / 4, 128, 0, stream>>>(logits, ldz, n_tokens, n_exp, top, score_kind, renormalize,
+                                                           expert_of, rank_of, weight_of, counts, correction, weight_scale, n_real, bias);
   FERRUM_CHECK_LAUNCH("moe_route");
   FERRUM_DISPATCH_DTYPE(dtype, T, (moe_gather_kernel<T><<<n_tokens * top, 128, 0, stream>>>(
       (const T*)x, ldx, E, n_real, top, expert_of, rank_of, weight_of, counts, scale_input, (T*)xg, row_of)));
@@ -669,13 +684,13 @@ FERRUM_API int ferrum_moe_gemm(const void* A, int lda, const void* W, int w_rows
 }
 
 FERRUM_API int ferrum_moe_combine(const float* rows, int ld, const int* row_of, const float* weight_of, int top, int n_tokens,
-                                  int E, float* y, const void* x, int ldx, int x_dtype, const float* add, int ld_add,
-                                  cudaStream_t stream) {
+                                  int E, float* y, const void* x, int ldx, int x_dtype, const float* add, int ld_add, int accumulate,
+                                  void* yc, int ldyc, cudaStream_t stream) {
   FERRUM_CHECK_ARG(top > 0 && E > 0 && ld >= E, "moe_combine: bad sizes");
-  FERRUM_CHECK_ARG((x == nullptr || ldx >= E) && (add == nullptr || ld_add >= E), "moe_combine: a row is shorter than the width");
+  FERRUM_CHECK_ARG((x == nullptr || ldx >= E) && (add == nullptr || ld_add >= E) && (yc == nullptr || ldyc >= E), "moe_combine: a row is shorter than the width");
   if (n_tokens == 0) return 0;
   FERRUM_DISPATCH_DTYPE(x_dtype, T, (moe_combine_kernel<T><<<n_tokens, 256, 0, stream>>>(rows, ld, row_of, weight_of, top, E, y,
-                                                                                       (const T*)x, ldx, add, ld_add)));
+                                                                                       (const T*)x, ldx, add, ld_add, accumulate, (T*)yc, ldyc)));
   FERRUM_CHECK_LAUNCH("moe_combine");
   return 0;
 }

@@ -5,8 +5,8 @@
 //                  the next sublayer reads (the sublayers of such a block read the residual row itself).  Without y
 //                  it only makes that copy (the first block's input).
 // dual_norm_mean:  out[t] = (rms(a[t]) * wa + rms(b[t]) * wb) / 2: two branches that read the same input meet.
-// head_gate_norm:  per (token, head): out = rms(o_head) * w * sigmoid(gate logits), rounded once to the compute
-//                  type; the weight is one vector for all heads or one per head.
+// head_gate_norm:  per (token, head): out = scale * rms(o_head) * w * g, with g = sigmoid or silu of the gate logits,
+//                  rounded once to the compute type; the weight is one vector for all heads or one per head.
 //
 // One block per token (one warp per token and head in head_gate_norm); a row's sums are taken with one fixed tree,
 // so a token's result does not depend on what else is in the batch.
@@ -61,7 +61,8 @@ dual_norm_mean_kernel(const float* __restrict__ a, int lda, const float* __restr
 template <typename T>
 __global__ void __launch_bounds__(128)
 head_gate_norm_kernel(const float* __restrict__ o, int ldo, const float* __restrict__ gate, int ldg, const float* __restrict__ w,
-                      int w_per_head, float eps, int n_tokens, int H, int Dv, T* __restrict__ out, int ldout) {
+                      int w_per_head, float eps, int n_tokens, int H, int Dv, T* __restrict__ out, int ldout, int gate_silu,
+                      float out_scale) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long item = (long long)blockIdx.x * 4 + warp;
   if (item >= (long long)n_tokens * H) return;
@@ -75,8 +76,8 @@ head_gate_norm_kernel(const float* __restrict__ o, int ldo, const float* __restr
   const float r = 1.f / sqrtf(ss / (float)Dv + eps);
   for (int d = lane; d < Dv; d += 32) {
     float v = src[d] * r * wr[d];
-    if (g != nullptr) v *= 1.f / (1.f + expf(-g[d]));
-    out[(size_t)t * ldout + (size_t)h * Dv + d] = from_f32<T>(v);
+    if (g != nullptr) v *= (gate_silu ? g[d] : 1.f) / (1.f + expf(-g[d]));
+    out[(size_t)t * ldout + (size_t)h * Dv + d] = from_f32<T>(v * out_scale);
   }
 }
 
@@ -101,15 +102,17 @@ FERRUM_API int ferrum_dual_norm_mean(const float* a, int lda, const float* b, in
 }
 
 // o float32 [T, >= H * Dv]; gate: float32 logits with the same layout and a stride of their own (may be null);
-// w: [Dv], or [H * Dv] with w_per_head; out [T, >= H * Dv] in the type `dtype`.
+// w: [Dv], or [H * Dv] with w_per_head; out [T, >= H * Dv] in the type `dtype`.  gate_silu: silu of the gate logits
+// instead of their sigmoid; out_scale multiplies every element.
 FERRUM_API int ferrum_head_gate_norm(const float* o, int ldo, const float* gate, int ldg, const float* w, int w_per_head, float eps,
-                                     int n_tokens, int H, int Dv, void* out, int ldout, int dtype, cudaStream_t stream) {
+                                     int n_tokens, int H, int Dv, void* out, int ldout, int dtype, int gate_silu, float out_scale,
+                                     cudaStream_t stream) {
   FERRUM_CHECK_ARG(H > 0 && Dv > 0 && ldo >= H * Dv && ldout >= H * Dv && (gate == nullptr || ldg >= H * Dv), "head_gate_norm: bad sizes");
   if (n_tokens == 0) return 0;
   const long long blocks = ((long long)n_tokens * H + 3) / 4;
   FERRUM_CHECK_ARG(blocks < (1LL << 31), "head_gate_norm: too many rows");
   FERRUM_DISPATCH_DTYPE(dtype, T, (head_gate_norm_kernel<T><<<(unsigned)blocks, 128, 0, stream>>>(o, ldo, gate, ldg, w, w_per_head, eps,
-                                                                                              n_tokens, H, Dv, (T*)out, ldout)));
+                                                                                              n_tokens, H, Dv, (T*)out, ldout, gate_silu, out_scale)));
   FERRUM_CHECK_LAUNCH("head_gate_norm");
   return 0;
 }

@@ -2,7 +2,8 @@
 
 The run order is data: `schedule` is a list of `Run(block, cache_of)`.  `block` indexes
 `blocks` (naming a block twice runs it twice, each run with cache planes of its own);
-`cache_of = j` lets run k read the cache that run j wrote instead of writing one.  The model
+`cache_of = j` lets run k read the cache that run j wrote instead of writing one; `before` names one of the
+model's `entries`, parts that rework the residual rows right before that run.  The model
 never looks at which architecture it is; `weight_specs` and `cache_needs` are derived from
 the parts.
 """
@@ -25,34 +26,38 @@ NVTX = os.environ.get("FERRUM_NVTX", "0") == "1"
 class Run:
     block: int
     cache_of: Optional[int] = None      # index of an earlier run whose cache this run reads
+    before: Optional[int] = None        # index into the model's `entries`: a part that runs on the residual rows first
 
 
 class DecoderModel(Part):
     graph_safe = True
 
     def __init__(self, config, dtype, embedding, position, blocks, final_norm, head, schedule=None,
-                 block_prefix="blk.{}.", names=("token_embd.", "output_norm.", "output."), shared=()):
+                 block_prefix="blk.{}.", names=("token_embd.", "output_norm.", "output."), shared=(), entries=()):
         """shared: (prefix, part) pairs the model owns because several blocks refer to them (a table
-        that every layer reads a slice of); they only bring parameters, the blocks call them."""
+        that every layer reads a slice of); they only bring parameters, the blocks call them.
+        entries: (prefix, part) pairs that runs of the schedule name in `before`."""
         self.config, self.dtype = config, dtype
         self.embedding, self.position, self.blocks = embedding, position, list(blocks)
         self.final_norm, self.head = final_norm, head
         self.schedule: List[Run] = list(schedule) if schedule is not None else [Run(i) for i in range(len(self.blocks))]
         self._block_prefix, self._names = block_prefix, names
-        self.shared = list(shared)
+        self.shared, self.entries = list(shared), list(entries)
         self.on_run = None       # debugging hook: called as on_run(k, h) after run k of the schedule with the residual rows
         for k, run in enumerate(self.schedule):
             if not 0 <= run.block < len(self.blocks):
                 raise ValueError(f"schedule entry {k} names block {run.block}, which does not exist")
             if run.cache_of is not None and not (0 <= run.cache_of < k and self.schedule[run.cache_of].cache_of is None):
                 raise ValueError(f"schedule entry {k} must read the cache of an earlier run that writes one")
+            if run.before is not None and not 0 <= run.before < len(self.entries):
+                raise ValueError(f"schedule entry {k} names entry part {run.before}, which does not exist")
 
     # ------------------------------------------------------------------ structure
     def children(self):
         out = [(self._names[0], self.embedding)]
         if self.position is not None:
             out.append(("position.", self.position))
-        out += self.shared
+        out += self.shared + self.entries
         out += [(self._block_prefix.format(i), b) for i, b in enumerate(self.blocks)]
         out += [(self._names[1], self.final_norm), (self._names[2], self.head)]
         return out
@@ -89,6 +94,8 @@ class DecoderModel(Part):
         for k, run in enumerate(self.schedule):
             if NVTX:
                 torch.cuda.nvtx.range_push(f"run {k} block {run.block}")
+            if run.before is not None:
+                self.entries[run.before][1].forward(h, ctx)
             self.blocks[run.block].forward(h, ctx, cache.layer_cache(k))
             if self.on_run is not None:
                 ctx.flush_residual()

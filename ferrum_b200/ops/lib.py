@@ -26,7 +26,7 @@ TC_STORE_BF16, TC_STORE_F32, TC_RESIDUAL, TC_SWIGLU, TC_GEGLU, TC_SWISH_CLAMP = 
 
 _lib = None
 _lock = threading.Lock()
-ABI = 17
+ABI = 18
 
 
 def lib():
@@ -231,6 +231,22 @@ def embedding(table, ids, out, err, scale=1.0, pos_table=None, positions=None, c
                                   c_int(V), _ptr(err), c_int(copies), _stream()), "embedding")
 
 
+def embedding_norm(table, ids, w, eps, out, err, copy=None):
+    """out[t] = rms(table[ids[t]]) * w, float32; copy (the table's type; may be a view into wider rows) receives it too."""
+    _need(table, None, "table", 2); _need(ids, torch.int32, "ids", 1); _need(out, torch.float32, "out", 2); _need(w, torch.float32, "w", 1)
+    V, E = table.shape
+    T = ids.shape[0]
+    if out.shape[0] < T or out.shape[1] != E or w.shape[0] != E or not table.is_contiguous() or not out.is_contiguous():
+        raise KernelError("embedding_norm: shapes do not agree")
+    if copy is not None:
+        _need(copy, table.dtype, "copy", 2)
+        if copy.shape[0] < T or copy.shape[1] < E:
+            raise KernelError("embedding_norm: the copy is too small")
+    _check(lib().ferrum_embedding_norm(_ptr(table), dtype_code(table.dtype), _ptr(ids), _ptr(w), c_float(eps), _ptr(out), _ptr(copy),
+                                       c_int(copy.stride(0) if copy is not None else 0), c_int(T), c_int(E), c_int(V), _ptr(err),
+                                       _stream()), "embedding_norm")
+
+
 class Partials:
     """A product that the tensor-core kernel left as float32 partials (see gemm_tc_deferred):
     the workspace that holds them and the four numbers a consumer needs to sum them."""
@@ -402,7 +418,7 @@ def attention_generic_split():
 
 def attention_generic(q, out, n_tokens, positions, req_of_token, block_table, kv_plane, page_stride, page_size, Hq,
                       Hkv, D, scale, window, err, part=None, split_slots=0, q_start=None, n_reqs=0, distance_penalty=None,
-                      chunked=False, softcap=0.0, sink=False):
+                      chunked=False, softcap=0.0, sink=False, keep_first=0, out_scale=1.0):
     """Causal GQA attention of every token over its request's pages on the CUDA cores, float32
     arithmetic.  part=None: one CTA per (token, group of heads) walks the whole key range (many
     tokens).  With `part` (float32, n_tokens * Hq * split_slots * (D + 2) elements) every row's keys
@@ -414,7 +430,9 @@ def attention_generic(q, out, n_tokens, positions, req_of_token, block_table, kv
     is taken off the scaled score; with r2 None it is the straight line r1[h] * (position - key position).
     chunked: `window` is the length of a chunk (positions are cut into chunks from 0; a query sees its own
     chunk's keys up to itself) instead of a sliding window.  softcap c > 0: the scaled score becomes c * tanh(score / c).
-    sink: a key of score 0 without a value joins every softmax (one more term in its denominator).  `out` may be float32 whatever the cache's type
+    sink: a key of score 0 without a value joins every softmax (one more term in its denominator).  keep_first: with a window,
+    the sequence's first so many keys are seen from everywhere; with `part`, split_slots must also cover their own
+    ceil(keep_first / split) splits.  out_scale multiplies the output.  `out` may be float32 whatever the cache's type
     (a kernel after this one still works on the heads' results)."""
     _need(q, None, "q", 2); _need(out, None, "out", 2); _need(kv_plane, q.dtype, "kv_plane")
     if out.dtype not in (q.dtype, torch.float32):
@@ -442,7 +460,8 @@ def attention_generic(q, out, n_tokens, positions, req_of_token, block_table, kv
                                           c_float(scale), c_int(window), _ptr(err), _ptr(part), c_int(split_slots),
                                           _ptr(q_start) if part is None else None, c_int(n_reqs), _ptr(r1), _ptr(r2),
                                           c_int(1 if out.dtype == torch.float32 and q.dtype != torch.float32 else 0),
-                                          c_int(1 if chunked else 0), c_float(softcap or 0.0), c_int(1 if sink else 0), _stream()),
+                                          c_int(1 if chunked else 0), c_float(softcap or 0.0), c_int(1 if sink else 0), c_int(int(keep_first)),
+                                          c_float(out_scale), _stream()),
            "attention_generic")
 
 
@@ -811,8 +830,8 @@ def qkv_shape(proj, n_tokens, ctx, block_table, rot, qk_pairing, value_rot, valu
            "qkv_shape")
 
 
-def attention_finish(o, n_tokens, ctx, value_rot, value_pairing, gate, out, Hq, Dv, Dp):
-    """out[t, h] = turn_back(o[t, h], position) * sigmoid(gate[t, h]) in the compute type; `value_rot`
+def attention_finish(o, n_tokens, ctx, value_rot, value_pairing, gate, out, Hq, Dv, Dp, out_scale=1.0):
+    """out[t, h] = out_scale * turn_back(o[t, h], position) * sigmoid(gate[t, h]) in the compute type; `value_rot`
     (None: no turn) and `gate` (float32 logits [T, Hq * Dv], may be a view into wider rows; None: no gate)."""
     _need(o, torch.float32, "o", 2); _need(out, None, "out", 2)
     if gate is not None:
@@ -822,7 +841,7 @@ def attention_finish(o, n_tokens, ctx, value_rot, value_pairing, gate, out, Hq, 
                                          c_int(value_pairing), c_int(value_rot.shape[0] if value_rot is not None else 0),
                                          _ptr(gate), c_int(gate.stride(0) if gate is not None else 0), _ptr(out),
                                          c_int(out.stride(0)), dtype_code(out.dtype), c_int(Hq), c_int(Dv), c_int(Dp),
-                                         _ptr(ctx.err), _stream()), "attention_finish")
+                                         _ptr(ctx.err), c_float(out_scale), _stream()), "attention_finish")
 
 
 # ----------------------------------------------------------------------------- state-space mixer
@@ -963,18 +982,18 @@ def hyper_step(X, S, E, n_rows, write=None, rows=None, store=True, in_w=None, no
 
 
 # ----------------------------------------------------------------------------- routed feed-forward
-MOE_SCORES = {"sigmoid": 0, "softmax": 1}
+MOE_SCORES = {"sigmoid": 0, "softmax": 1, "chosen_softmax": 2}      # chosen_softmax: the logits choose, the weights are a softmax over the chosen
 
 
 MOE_MAX_EXPERTS, MOE_MAX_TOP = 256, 8      # (the routing kernel's own limits, which it checks again)
 
 
 def moe_route(logits, n_tokens, n_exp, top, x, scale_input, expert_of, rank_of, weight_of, counts, xg, row_of, scores="sigmoid",
-              renormalize=False, correction=None, weight_scale=1.0, n_identity=0):
+              renormalize=False, correction=None, weight_scale=1.0, n_identity=0, bias=None):
     """From the router's float32 logits [T, >= n_exp]: every token's `top` experts and their weights, and the
     tokens' input rows x [T, E] gathered into xg [T * top, E] sorted by expert (times the weight when
     `scale_input`); row_of [T * top] says where each (token, choice) went; counts [n_exp] the rows per expert.
-    correction (float32 [n_exp]) is added to the scores for the choice only; the weights are the plain scores times
+    bias (float32 [n_exp]) is added to the logits first.  correction (float32 [n_exp]) is added to the scores for the choice only; the weights are the plain scores times
     weight_scale.  The last n_identity of the n_exp router outputs are identity experts: they get no rows (row_of -1)."""
     global launches
     _need(logits, torch.float32, "logits", 2); _need(x, None, "x", 2); _need(xg, x.dtype, "xg", 2)
@@ -984,15 +1003,16 @@ def moe_route(logits, n_tokens, n_exp, top, x, scale_input, expert_of, rank_of, 
     E = x.shape[1]
     if xg.shape[1] != E or xg.shape[0] < n_tokens * top or not xg.is_contiguous() or counts.numel() < n_exp - n_identity:
         raise KernelError("moe_route: buffers are too small")
-    if correction is not None:
-        _need(correction, torch.float32, "correction", 1)
-        if correction.shape[0] != n_exp or not correction.is_contiguous():
-            raise KernelError("moe_route: the correction has one number per router output")
+    for v, what in ((correction, "correction"), (bias, "bias")):
+        if v is not None:
+            _need(v, torch.float32, what, 1)
+            if v.shape[0] != n_exp or not v.is_contiguous():
+                raise KernelError(f"moe_route: the {what} has one number per router output")
     _check(lib().ferrum_moe_route(_ptr(logits), c_int(logits.stride(0)), c_int(n_tokens), c_int(n_exp), c_int(top),
                                   c_int(MOE_SCORES[scores]), c_int(1 if renormalize else 0), _ptr(x), c_int(x.stride(0)), c_int(E),
                                   dtype_code(x.dtype), c_int(1 if scale_input else 0), _ptr(expert_of), _ptr(rank_of),
                                   _ptr(weight_of), _ptr(counts), _ptr(xg), _ptr(row_of), _ptr(correction), c_float(weight_scale),
-                                  c_int(n_identity), _stream()), "moe_route")
+                                  c_int(n_identity), _ptr(bias), _stream()), "moe_route")
     launches += 1          # (the entry point launches the routing and the gather)
 
 
@@ -1036,10 +1056,11 @@ def set_moe_cuda_cores(on: bool):
     lib().ferrum_moe_cuda_cores(c_int(1 if on else 0))
 
 
-def moe_combine(rows, row_of, top, n_tokens, y, weight_of=None, x=None, add=None):
+def moe_combine(rows, row_of, top, n_tokens, y, weight_of=None, x=None, add=None, accumulate=False, copy=None):
     """y[t] = sum_j rows[row_of[t, j]] (times weight_of[t, j] when given), float32.  x [T, E] (any type): the tokens'
     own input rows, which stand in for choices without a row (row_of < 0: identity experts); add (float32 [T, E]): rows
-    that join the sum last."""
+    that join the sum last.  accumulate: y gains the sum; copy (a compute-type buffer, x's type when both are given): receives
+    the new y."""
     _need(rows, torch.float32, "rows", 2); _need(y, torch.float32, "y", 2); _need(row_of, torch.int32, "row_of")
     E = y.shape[1]
     if not y.is_contiguous() or rows.shape[1] < E:
@@ -1048,12 +1069,15 @@ def moe_combine(rows, row_of, top, n_tokens, y, weight_of=None, x=None, add=None
         _need(x, None, "x", 2)
     if add is not None:
         _need(add, torch.float32, "add", 2)
-    if (x is not None and x.shape[1] < E) or (add is not None and add.shape[1] < E):
+    if copy is not None:
+        _need(copy, x.dtype if x is not None else None, "copy", 2)
+    if any(t is not None and t.shape[1] < E for t in (x, add, copy)):
         raise KernelError("moe_combine: shapes do not agree")
     _check(lib().ferrum_moe_combine(_ptr(rows), c_int(rows.stride(0)), _ptr(row_of), _ptr(weight_of), c_int(top), c_int(n_tokens),
                                     c_int(E), _ptr(y), _ptr(x), c_int(x.stride(0) if x is not None else 0),
-                                    dtype_code(x.dtype) if x is not None else c_int(F32), _ptr(add),
-                                    c_int(add.stride(0) if add is not None else 0), _stream()), "moe_combine")
+                                    dtype_code(x.dtype if x is not None else copy.dtype if copy is not None else torch.float32), _ptr(add),
+                                    c_int(add.stride(0) if add is not None else 0), c_int(1 if accumulate else 0), _ptr(copy),
+                                    c_int(copy.stride(0) if copy is not None else 0), _stream()), "moe_combine")
 
 
 def softcap(x, n_rows, cap):
@@ -1098,8 +1122,9 @@ def dual_norm_mean(a, b, wa, wb, eps, out, n_tokens):
                                        c_int(E), _ptr(out), c_int(out.stride(0)), c_int(n_tokens), _stream()), "dual_norm_mean")
 
 
-def head_gate_norm(o, gate, w, eps, n_tokens, H, Dv, out):
-    """out[t, h] = rms(o[t, h]) * w * sigmoid(gate[t, h]) per head of Dv elements, rounded once to out's type.  o, gate:
+def head_gate_norm(o, gate, w, eps, n_tokens, H, Dv, out, gate_act="sigmoid", out_scale=1.0):
+    """out[t, h] = out_scale * rms(o[t, h]) * w * g per head of Dv elements with g = sigmoid(gate[t, h]), or silu of it
+    (gate_act), rounded once to out's type.  o, gate:
     float32 rows (gate may be a view into wider rows, or None); w: float32 [Dv] (one for all heads) or [H * Dv]."""
     _need(o, torch.float32, "o", 2); _need(out, None, "out", 2); _need(w, torch.float32, "w", 1)
     if gate is not None:
@@ -1109,7 +1134,8 @@ def head_gate_norm(o, gate, w, eps, n_tokens, H, Dv, out):
     _bytes_work((o, n_tokens), (gate, n_tokens), (out, n_tokens))
     _check(lib().ferrum_head_gate_norm(_ptr(o), c_int(o.stride(0)), _ptr(gate), c_int(gate.stride(0) if gate is not None else 0),
                                        _ptr(w), c_int(1 if w.shape[0] == H * Dv and H > 1 else 0), c_float(eps), c_int(n_tokens),
-                                       c_int(H), c_int(Dv), _ptr(out), c_int(out.stride(0)), dtype_code(out.dtype), _stream()),
+                                       c_int(H), c_int(Dv), _ptr(out), c_int(out.stride(0)), dtype_code(out.dtype),
+                                       c_int({"sigmoid": 0, "silu": 1}[gate_act]), c_float(out_scale), _stream()),
            "head_gate_norm")
 
 
@@ -1174,3 +1200,82 @@ def matrix_memory(proj, offsets, bias_i, bias_f, cap, n_tokens, ctx, H, D, Dv, s
                                       _ptr(ctx.slots), c_int(H), c_int(D), c_int(Dv), _ptr(state), c_longlong(state.stride(0)),
                                       _ptr(gates), _ptr(o), c_int(o.stride(0)), _stream()), "matrix_memory")
     launches += 1          # (the entry point launches the gates and the walk)
+
+
+# ----------------------------------------------------------------------------- decays per key channel
+def channel_decay_segments(ctx, H, D, Dv):
+    """(tokens per segment, segments) of the step's walk: (0, 0) while no portion is worth cutting.  Portions are cut so that
+    about as many blocks run at a time as the GPU holds; single tokens (and so every captured step) are never cut."""
+    longest = ctx.max_q_len
+    if longest < CHANNEL_DECAY_CUT_FROM:
+        return 0, 0
+    cols = int(lib().ferrum_channel_decay_block_columns(c_int(D), c_int(Dv)))
+    per_segment = H * -(-Dv // cols)                       # blocks of one segment
+    length = -(-ctx.n_tokens * per_segment // (CHANNEL_DECAY_BLOCKS_PER_SM * sm_count()))
+    length = max(CHANNEL_DECAY_MIN_SEGMENT, -(-length // 16) * 16)
+    if longest <= length:
+        return 0, 0
+    return length, sum(-(-n // length) for n in ctx.h_q_len)
+
+
+CHANNEL_DECAY_CUT_FROM, CHANNEL_DECAY_MIN_SEGMENT, CHANNEL_DECAY_BLOCKS_PER_SM = 48, 32, 3
+
+
+def channel_decay(q, k, v, dec, n_tokens, ctx, H, D, Dv, state, o, bonus=None, out_scale=1.0, segments=None):
+    """The walk of a recurrence whose state rows decay per key channel (see csrc/kernels/channel_decay.cu).  q, k, dec: float32
+    rows [T, >= H D]; v: [T, >= H Dv] (views into wider rows are fine); state: float32 [max_requests, >= H D Dv], a row's first
+    H D Dv floats are S; o: float32 [T, H Dv].  bonus (float32 [H, D]): the current token enters the read-out through it, before
+    the write; without it the read-out follows the write.  segments: (length, number) instead of `channel_decay_segments`'."""
+    global launches
+    for t, n, w in ((q, "q", H * D), (k, "k", H * D), (v, "v", H * Dv), (dec, "dec", H * D), (o, "o", H * Dv), (state, "state", H * D * Dv)):
+        _need(t, torch.float32, n, 2)
+        if t.shape[1] < w or (n != "state" and t.shape[0] < n_tokens):
+            raise KernelError(f"channel_decay: {n} is too small")
+    if bonus is not None:
+        _need(bonus, torch.float32, "bonus")
+        if bonus.numel() != H * D or not bonus.is_contiguous():
+            raise KernelError("channel_decay: the bonus has one number per head and key channel")
+    length, n_seg = channel_decay_segments(ctx, H, D, Dv) if segments is None else segments
+    seg_state = seg_dec = None
+    if length:
+        seg_state = ctx.buf("cdecay_seg_state", (n_seg * H * D * Dv,), torch.float32)
+        seg_dec = ctx.buf("cdecay_seg_dec", (n_seg * H * D,), torch.float32)
+    if _profile is not None:
+        global _work
+        _work = (4 * (n_tokens * (3 * H * D + 2 * H * Dv) + 2 * ctx.n_reqs * H * D * Dv), 5.0 * n_tokens * H * D * Dv)
+    _check(lib().ferrum_channel_decay(_ptr(q), c_int(q.stride(0)), _ptr(k), c_int(k.stride(0)), _ptr(v), c_int(v.stride(0)), _ptr(dec),
+                                      c_int(dec.stride(0)), _ptr(bonus), c_float(out_scale), c_int(n_tokens), c_int(ctx.n_reqs),
+                                      _ptr(ctx.q_start), _ptr(ctx.slots), c_int(H), c_int(D), c_int(Dv), _ptr(state),
+                                      c_longlong(state.stride(0)), c_int(length), c_int(n_seg), _ptr(seg_state), _ptr(seg_dec), _ptr(o),
+                                      c_int(o.stride(0)), _stream()), "channel_decay")
+    launches += 2 if length else 0         # (the segments' contributions, their chain, the walk)
+
+
+def channel_decay_gate(low, w2, bias, kind, n_tokens, out, tanh=False, tau=1.0):
+    """out[t, n] = f(sum_r w2[n, r] act(low[t, r]) + bias[n]) in float32: kind "exp_exp": f(z) = exp(-exp(z)); "sigmoid_root":
+    f(z) = sigmoid(z)^(1/tau).  act: the identity or tanh.  low: float32 [T, rank] (may be a view); w2: compute type."""
+    _need(low, torch.float32, "low", 2); _need(w2, None, "w2", 2); _need(bias, torch.float32, "bias", 1); _need(out, torch.float32, "out", 2)
+    N, rank = w2.shape
+    if low.shape[1] < rank or bias.shape[0] != N or out.shape[1] < N or not w2.is_contiguous() or min(low.shape[0], out.shape[0]) < n_tokens:
+        raise KernelError("channel_decay_gate: shapes do not agree")
+    _bytes_work((low, n_tokens), (out, n_tokens), (w2, N))
+    _check(lib().ferrum_channel_decay_gate(_ptr(low), c_int(low.stride(0)), c_int(rank), c_int(1 if tanh else 0), _ptr(w2), dtype_code(w2.dtype),
+                                           _ptr(bias), c_int({"exp_exp": 0, "sigmoid_root": 1}[kind]), c_float(1.0 / tau), c_int(n_tokens),
+                                           c_int(N), _ptr(out), c_int(out.stride(0)), _stream()), "channel_decay_gate")
+
+
+def token_shift_mix(x, mu, n_tokens, ctx, prev, out, counts=None):
+    """out[m, t] = x[t] + (x of the request's token before - x[t]) * mu[m], rounded once to x's type; x [T, E]; mu: float32
+    [n, E]; prev: float32 [max_requests, E] view of the requests' state rows (read at a portion's first token, and the
+    portion's last row is left there); out: [n, T, E] contiguous.  counts (int32): filled with n_tokens."""
+    _need(x, None, "x", 2); _need(mu, torch.float32, "mu", 2); _need(prev, torch.float32, "prev", 2); _need(out, x.dtype, "out", 3)
+    n, E = mu.shape
+    if x.shape[1] != E or prev.shape[1] != E or tuple(out.shape) != (n, n_tokens, E) or not out.is_contiguous() or not mu.is_contiguous():
+        raise KernelError("token_shift_mix: shapes do not agree")
+    if counts is not None:
+        _need(counts, torch.int32, "counts", 1)
+    _bytes_work((x, 2 * n_tokens), (out, n * n_tokens))
+    _check(lib().ferrum_token_shift_mix(_ptr(x), c_int(x.stride(0)), dtype_code(x.dtype), c_int(E), _ptr(mu), c_int(n), _ptr(ctx.q_start),
+                                        _ptr(ctx.req_of_token), _ptr(ctx.slots), _ptr(prev), c_longlong(prev.stride(0)), _ptr(out),
+                                        c_int(n_tokens), _ptr(counts), c_int(counts.shape[0] if counts is not None else 0), _stream()),
+           "token_shift_mix")

@@ -47,6 +47,7 @@ class PagedAttention(Mixer):
         self.position, self.dtype, self.window = position, dtype, int(window)
         self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(head_dim)
         self.chunked = False     # True: `window` is a chunk length (a subclass sets it)
+        self.keep_first = 0      # with a window: the sequence's first keys that every query sees (a subclass sets it)
         self.score_softcap, self.sink = 0.0, False      # (a subclass may bend the scores and add a sink to the softmax)
         self.w_q_weight = self.w_k_weight = self.w_v_weight = self.w_output_weight = None
         self.w_qkv = None
@@ -85,7 +86,7 @@ class PagedAttention(Mixer):
             self._generic(qkv, out, ctx, cache, table)
         linear(out, self.w_output_weight, residual, RESIDUAL if accumulate else STORE_F32, ctx, M=T)
 
-    def _generic(self, qkv, out, ctx, cache, table, distance_penalty=None):
+    def _generic(self, qkv, out, ctx, cache, table, distance_penalty=None, out_scale=1.0):
         """CUDA-core path.  With enough rows to fill the GPU (a prompt portion) every row walks its
         keys alone; with few (decoding) the keys of a row are cut into splits among CTAs.  Which of
         the two runs depends on the number of tokens only, and so does the number of split slots
@@ -99,12 +100,12 @@ class PagedAttention(Mixer):
             longest = table.shape[1] * cache.page_size if ctx.fixed_shapes else ctx.max_kv_len
             if self.window > 0:
                 longest = min(longest, self.window + split)       # a window of w keys touches at most w / split + 2 splits
-            slots = longest // split + 2
+            slots = longest // split + 2 + (-(-self.keep_first // split) if self.window > 0 else 0)
             part = ctx.buf("attn_generic_part", (T * Hq * slots * (D + 2),), torch.float32)
         ops.attention_generic(qkv, out, T, ctx.positions, ctx.req_of_token, table, cache.plane, cache.page_stride,
                               cache.page_size, Hq, Hkv, D, self.scale, self.window, ctx.err, part, slots,
                               q_start=ctx.q_start, n_reqs=ctx.n_reqs, distance_penalty=distance_penalty, chunked=self.chunked,
-                              softcap=self.score_softcap, sink=self.sink)
+                              softcap=self.score_softcap, sink=self.sink, keep_first=self.keep_first, out_scale=out_scale)
 
     def plan(self, ctx, cache):
         """The step's work lists of the tensor-core kernels for this layer's shape (None on the

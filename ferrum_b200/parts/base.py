@@ -54,11 +54,13 @@ class ParamSpec:
 class PagedKVNeed:
     """Keys and values of `n_kv_heads` x `head_dim` per position; `window` 0 keeps all keys.
     `parts` 2: a page holds keys, then values; 1: one row per position and head (a mixer that
-    derives keys and values from the same cached row)."""
+    derives keys and values from the same cached row).  `keep_first`: with a window, the first so many
+    positions stay for the whole sequence."""
     n_kv_heads: int
     head_dim: int
     window: int = 0
     parts: int = 2
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)

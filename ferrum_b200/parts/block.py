@@ -1,4 +1,6 @@
-"""A pre-norm block: h += mixer(norm1(h)); h += ffn(norm2(h)).
+"""Blocks: how a layer's norms, mixer and feed-forward meet the residual stream.
+
+`PreNormBlock`: h += mixer(norm1(h)); h += ffn(norm2(h)).
 
 The reference's order (crates/model/src/llama.rs:183-285; docs/ARCHITECTURE.md "Forward
 pass").  The two residual sums happen inside the parts' last kernels, in float32.
@@ -9,27 +11,68 @@ import torch
 
 from ..ops import lib as ops
 from .base import CacheNeed, FeedForward, Mixer, Norm, ParamSpec, Part, StateNeed
+from .ffn import RoutedFeedForward
 from .linear import STORE_F32, linear, linear_deferred
 
 
 class PreNormBlock(Part):
+    """h += mixer(norm1(h)); h += ffn(norm2(h)); then, when the block has one, a `TokenSideInput` adds its
+    token-dependent branch.  `ffn` (with norm2) may be None.  A routed feed-forward leaves the new rows in the
+    compute type on the way, for the side input's product."""
     graph_safe = True
 
-    def __init__(self, norm1: Norm, mixer: Mixer, norm2: Norm, ffn: FeedForward,
-                 names=("attn_norm.", "attn_", "ffn_norm.", "ffn_")):
-        self.norm1, self.mixer, self.norm2, self.ffn = norm1, mixer, norm2, ffn
+    def __init__(self, norm1: Norm, mixer: Mixer, norm2: Norm = None, ffn: FeedForward = None,
+                 names=("attn_norm.", "attn_", "ffn_norm.", "ffn_", "side."), side: "TokenSideInput" = None):
+        if (norm2 is None) != (ffn is None):
+            raise ValueError("the second norm and the feed-forward come together")
+        self.norm1, self.mixer, self.norm2, self.ffn, self.side = norm1, mixer, norm2, ffn, side
         self._names = names
 
     def children(self):
-        return list(zip(self._names, (self.norm1, self.mixer, self.norm2, self.ffn)))
+        parts = (self.norm1, self.mixer, self.norm2, self.ffn, self.side)
+        return [(n, p) for n, p in zip(self._names, parts) if p is not None]
 
     def forward(self, h, ctx, cache):
         x = self.norm1.forward(h, ctx)
         ctx.flush_residual()            # no-op when the norm took the pending sum itself
         self.mixer.forward(x, ctx, cache, h)
-        x = self.norm2.forward(h, ctx)
+        rows = h                        # what the side input's product reads
+        if self.side is not None and self.side.dtype != torch.float32:
+            rows = ctx.buf("side_rows", (ctx.token_capacity, h.shape[1]), self.side.dtype)
+        copied = rows is h
+        if self.ffn is not None:
+            x = self.norm2.forward(h, ctx)
+            ctx.flush_residual()
+            if isinstance(self.ffn, RoutedFeedForward):
+                self.ffn.forward(x, ctx, h, copy=None if copied else rows)
+                copied = True
+            else:
+                self.ffn.forward(x, ctx, h)
+        if self.side is not None:
+            ctx.flush_residual()
+            if not copied:
+                ops.post_norm_add(h, ctx.n_tokens, xc=rows)
+            self.side.forward(h, rows, ctx, 1.0)
+
+
+class RestartInput(Part):
+    """What a pass of a looped range of layers starts with: h <- W [h; x0], x0 being the embedding's output.  The two lie
+    side by side in the step's buffer `restart_rows` (compute type): the embedding fills the second half
+    (`TokenEmbedding(restart=True)`) and this part the first."""
+    graph_safe = True
+
+    def __init__(self, width, dtype):
+        self.width, self.dtype = width, dtype
+        self.w_weight = None
+
+    def param_specs(self):
+        return {"weight": ParamSpec((self.width, 2 * self.width))}
+
+    def forward(self, h, ctx):
         ctx.flush_residual()
-        self.ffn.forward(x, ctx, h)
+        rows = ctx.buf("restart_rows", (ctx.token_capacity, 2 * self.width), self.dtype)
+        ops.post_norm_add(h, ctx.n_tokens, xc=rows[:, :self.width])
+        linear(rows, self.w_weight, h, STORE_F32, ctx, M=ctx.n_tokens)
 
 
 class PostNormBlock(Part):

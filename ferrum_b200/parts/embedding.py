@@ -18,23 +18,42 @@ from .linear import STORE_F32, linear
 class TokenEmbedding(Part):
     graph_safe = True
 
-    def __init__(self, n_vocab, width, scale=1.0, positions: "LearnedPositions" = None, copies=1, copy_dtype=None):
+    def __init__(self, n_vocab, width, scale=1.0, positions: "LearnedPositions" = None, copies=1, copy_dtype=None,
+                 norm=None, restart_dtype=None):
         """positions: a `LearnedPositions` part whose vector for a token's position is added to the
         (scaled) embedding; the model lists it as its position encoding, which owns the table.
         copies > 1: the residual rows are [tokens, copies * width], every copy the embedded token (a
         model whose blocks keep several residual streams).  copy_dtype (a 16-bit type): the rows are also left
         in that type in the step's buffer `residual_copy`, for blocks whose sublayers read the residual row
-        itself (`PostNormBlock`, which keeps the copy up to date)."""
+        itself (`PostNormBlock`, which keeps the copy up to date).  norm (an `RMSNorm`, whose parameters are named
+        `norm.`): the embedded row passes it before anything else.  restart_dtype: the row (after the norm) is also left in
+        that type in the second half of the step's buffer `restart_rows` (see `RestartInput`)."""
         self.n_vocab, self.width, self.scale, self.positions = n_vocab, width, float(scale), positions
         self.copies = int(copies)
+        self.norm, self.restart_dtype = norm, restart_dtype
+        if norm is not None and (self.scale != 1.0 or positions is not None or self.copies != 1):
+            raise ValueError("a normed embedding is neither scaled nor positioned and has one copy")
+        if restart_dtype is not None and norm is None:
+            raise ValueError("the restart rows are filled by the embedding's norm")
         self.copy_dtype = copy_dtype if copy_dtype not in (None, torch.float32) else None
         self.w_weight = None
 
     def param_specs(self):
         return {"weight": ParamSpec((self.n_vocab, self.width))}
 
+    def children(self):
+        return [("norm.", self.norm)] if self.norm is not None else []
+
     def forward(self, ctx):
         h = ctx.buf("hidden", (ctx.token_capacity, self.copies * self.width), torch.float32)
+        if self.norm is not None:
+            restart = None
+            if self.restart_dtype is not None:
+                restart = ctx.buf("restart_rows", (ctx.token_capacity, 2 * self.width), self.restart_dtype)[:, self.width:]
+            ops.embedding_norm(self.w_weight, ctx.token_ids, self.norm.w_weight, self.norm.eps, h, ctx.err, copy=restart)
+            if self.copy_dtype is not None:
+                ops.post_norm_add(h, ctx.n_tokens, xc=ctx.buf("residual_copy", (ctx.token_capacity, self.width), self.copy_dtype))
+            return h
         pos = self.positions.w_weight if self.positions is not None else None
         ops.embedding(self.w_weight, ctx.token_ids, h, ctx.err, scale=self.scale, pos_table=pos,
                       positions=ctx.positions if pos is not None else None, copies=self.copies)

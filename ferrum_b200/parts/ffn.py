@@ -113,7 +113,9 @@ class RoutedFeedForward(FeedForward):
     down_e(act(gate_e z) * (up_e z)), chosen by a router.
 
     router logits   W_router x in float32 (x in the compute type)
-    scores          "sigmoid" of each logit, or "softmax" over all experts
+    router_bias     a vector added to the logits
+    scores          "sigmoid" of each logit, "softmax" over all experts, or "chosen_softmax": the logits choose and
+                    the weights are a softmax over the chosen ones only
     choice          the `top` largest scores (a tie goes to the lower index)
     weights         the chosen scores, divided by their sum when `renormalize`
     scale_input     True: an expert sees z = weight * x and its result is added as it is;
@@ -129,11 +131,12 @@ class RoutedFeedForward(FeedForward):
     the activation, then down) run over it with the experts' stacked matrices, every CTA finding its
     expert from per-expert counters on the device, so a step's launches depend on the batch's sizes
     only.  `forward_rows` hands the unsummed result rows to a block that adds them itself;
-    `forward(accumulate=False)` sums them into the block's buffer."""
+    `forward` adds their sum to the residual rows, or (accumulate=False) leaves it in the block's buffer."""
     graph_safe = True
 
     def __init__(self, width, hidden, n_experts, top, dtype, act="silu", scores="sigmoid", renormalize=False, scale_input=True,
-                 correction=False, weight_scale=1.0, identity=0, limit=0.0, shared: FeedForward = None):
+                 correction=False, weight_scale=1.0, identity=0, limit=0.0, shared: FeedForward = None,
+                 router_bias=False):
         if act not in ops.GLU_ACTS:
             raise ValueError(f"unknown activation {act!r}")
         if scores not in ops.MOE_SCORES:
@@ -148,13 +151,16 @@ class RoutedFeedForward(FeedForward):
             raise ValueError("the clamped unit needs a positive limit")
         self.has_correction, self.weight_scale, self.identity = bool(correction), float(weight_scale), identity
         self.limit, self.shared = float(limit), shared
-        self.w_correction = None
+        self.has_router_bias = bool(router_bias)
+        self.w_correction = self.w_router_bias = None
         self.width, self.hidden, self.n_experts, self.top, self.dtype = width, hidden, int(n_experts), int(top), dtype
         self.act, self.scores, self.renormalize, self.scale_input = act, scores, bool(renormalize), bool(scale_input)
         self.w_router_weight = self.w_gate_up = self.w_down = None
 
     def param_specs(self):
         out = {"router.weight": ParamSpec((self.n_experts + self.identity, self.width))}
+        if self.has_router_bias:
+            out["router.bias"] = ParamSpec((self.n_experts + self.identity,), kind="vector", init="normal")
         if self.has_correction:
             out["correction"] = ParamSpec((self.n_experts + self.identity,), kind="vector", init="normal")
         for e in range(self.n_experts):
@@ -192,7 +198,7 @@ class RoutedFeedForward(FeedForward):
         xg = ctx.buf("moe_x", (cap * top, self.width), self.dtype)
         ops.moe_route(logits, T, n_out, top, x, self.scale_input, expert_of, rank_of, weight_of, counts, xg, row_of,
                       scores=self.scores, renormalize=self.renormalize, correction=self.w_correction if self.has_correction else None,
-                      weight_scale=self.weight_scale, n_identity=self.identity)
+                      weight_scale=self.weight_scale, n_identity=self.identity, bias=self.w_router_bias if self.has_router_bias else None)
         act = ctx.buf("moe_act", (cap * top, self.hidden), self.dtype)
         ops.moe_gemm(xg, self.w_gate_up, counts, T * top, act, self.hidden, glu=self.act, err=ctx.err, limit=self.limit)
         rows = ctx.buf("moe_rows", (cap * top, self.width), torch.float32)
@@ -200,9 +206,8 @@ class RoutedFeedForward(FeedForward):
         self._weight_of = weight_of
         return rows, row_of, top
 
-    def forward(self, x, ctx, residual, accumulate=True, defer=False):
-        if accumulate:
-            raise ValueError("a routed feed-forward hands its result to a block that adds it")
+    def forward(self, x, ctx, residual, accumulate=True, defer=False, copy=None):
+        """copy (a compute-type buffer [T, width]): also receives the new rows of `residual`."""
         add = join = None
         if self.shared is not None:
             add = ctx.buf("moe_shared", (ctx.token_capacity, self.width), torch.float32)
@@ -229,5 +234,5 @@ class RoutedFeedForward(FeedForward):
         if join is not None:
             torch.cuda.current_stream().wait_event(join)
         ops.moe_combine(rows, row_of, top, ctx.n_tokens, residual, weight_of=None if self.scale_input else self._weight_of,
-                        x=x if self.identity else None, add=add)
+                        x=x if self.identity else None, add=add, accumulate=accumulate, copy=copy)
         return None

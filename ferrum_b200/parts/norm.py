@@ -1,6 +1,7 @@
 """RMSNorm: x * rsqrt(mean(x^2) + eps) * w (crates/kernels/src/scalar.rs:143-156).  With
 `groups` > 1 the row is cut into that many equal consecutive parts, each divided by its own root
-mean square (the reference has one group)."""
+mean square (the reference has one group).  `zero_centred`: the file stores the weight around zero and
+the norm multiplies by 1 + w."""
 from __future__ import annotations
 
 from ..ops import lib as ops
@@ -10,14 +11,19 @@ from .base import Norm, ParamSpec
 class RMSNorm(Norm):
     graph_safe = True
 
-    def __init__(self, width: int, eps: float, out_dtype, groups: int = 1):
+    def __init__(self, width: int, eps: float, out_dtype, groups: int = 1, zero_centred: bool = False):
         if groups < 1 or width % groups:
             raise ValueError(f"{groups} groups do not divide a width of {width}")
         self.width, self.eps, self.out_dtype, self.groups = width, float(eps), out_dtype, int(groups)
+        self.zero_centred = bool(zero_centred)
         self.w_weight = None
 
     def param_specs(self):
-        return {"weight": ParamSpec((self.width,), kind="vector", init="ones_normal")}
+        return {"weight": ParamSpec((self.width,), kind="vector", init="normal" if self.zero_centred else "ones_normal")}
+
+    def finalize(self):
+        if self.zero_centred:
+            self.w_weight = 1.0 + self.w_weight          # (a float32 vector: the kernels see a plain weight)
 
     def forward(self, h, ctx, rows=None, n_rows=None, tag="norm"):
         """h float32 [T, width] -> compute-dtype rows; `rows` (int32) picks source rows."""

@@ -12,6 +12,8 @@ What a configuration may switch on, each with its constants as parameters:
   window         a query sees itself and the window - 1 keys before it (0: all); with mask="chunk"
                  positions are cut into chunks of `window` from position 0 and a query sees the keys of
                  its own chunk up to itself
+  keep_first     beside its window a query sees the sequence's first keep_first keys (whose pages the cache then
+                 never gives back before the request ends)
   dim != vdim    key and value heads of different sizes share pages of max(dim, vdim)-element rows
   qkv_bias       q, k and v projections have bias vectors
   qk_norm        every q and k head is divided by its root mean square and multiplied by a weight
@@ -53,8 +55,9 @@ class ShapedAttention(PagedAttention):
     def __init__(self, width, n_head, n_head_kv, dim, vdim, dtype, scale, eps=1e-6, window=0, rotary=None, unit_norm=False,
                  value_rotary=None, distance_penalty=False, gate=False, mask="window", qkv_bias=False, qk_norm=False,
                  query_temperature=None, linear_bias=None, value_mix=None, value_mix_key="v_first", value_from_key=False,
-                 score_softcap=0.0, sink=False):
+                 score_softcap=0.0, sink=False, keep_first=0):
         super().__init__(width, n_head, n_head_kv, max(int(dim), int(vdim)), rotary, dtype, window=window, scale=scale)
+        self.keep_first = int(keep_first) if self.window > 0 else 0
         self.score_softcap, self.sink = float(score_softcap or 0.0), bool(sink)
         self.value_from_key = bool(value_from_key)
         if self.value_from_key and (int(dim) != int(vdim) or qkv_bias or value_rotary is not None or value_mix is not None):
@@ -126,12 +129,23 @@ class ShapedAttention(PagedAttention):
             self.w_vmix = self.w_vmix.reshape(1).contiguous()
 
     def cache_need(self):
-        return CacheNeed(paged=PagedKVNeed(self.Hkv, self.D, self.window))
+        return CacheNeed(paged=PagedKVNeed(self.Hkv, self.D, self.window, keep_first=self.keep_first))
 
     def plan(self, ctx, cache):
         return None
 
-    def forward(self, x, ctx, cache, residual, accumulate=True, defer=False):
+    @property
+    def heads_width(self):
+        return self.Hq * self.Dv
+
+    def take_output_weight(self):
+        """The output matrix, for an owner that makes the output product itself (see `forward_heads`)."""
+        w, self.w_output_weight = self.w_output_weight, None
+        return w
+
+    def forward_heads(self, x, ctx, cache, out, scale=1.0):
+        """The heads' results side by side, times `scale`, into out [T, heads_width] (compute type; may be a view into
+        wider rows): everything but the output product."""
         T, Hq, Hkv, Dk, Dv, Dp = ctx.n_tokens, self.Hq, self.Hkv, self.Dk, self.Dv, self.D
         cap = ctx.token_capacity
         proj = ctx.buf("sattn_proj", (cap, self.w_in.shape[0]), torch.float32)
@@ -150,14 +164,18 @@ class ShapedAttention(PagedAttention):
                       k_norm=self.w_k_norm_weight if self.qk_norm else None, q_temp=self.q_temp, value_mix=mix,
                       whole_norm=self.whole_norm, value_from_key=self.value_from_key)
         penalty = (self.w_r1, self.w_r2) if self.has_penalty else ((self.slopes, None) if self.slopes is not None else None)
-        out = ctx.buf("sattn_out", (cap, Hq * Dv), self.dtype)
         if Dp == Dv and vrot is None and not self.has_gate:
             # nothing is left to do to the heads' results: the attention kernel rounds its float32 sums once into `out`
-            self._generic(q, out, ctx, cache, table, penalty)
+            self._generic(q, out, ctx, cache, table, penalty, out_scale=scale)
         else:
             o = ctx.buf("sattn_o", (cap, Hq * Dp), torch.float32)
             self._generic(q, o, ctx, cache, table, penalty)
-            self._finish(o, out, proj, ctx, vrot)
+            self._finish(o, out, proj, ctx, vrot, scale)
+
+    def forward(self, x, ctx, cache, residual, accumulate=True, defer=False):
+        T = ctx.n_tokens
+        out = ctx.buf("sattn_out", (ctx.token_capacity, self.heads_width), self.dtype)
+        self.forward_heads(x, ctx, cache, out)
         if defer and not accumulate:
             part = linear_deferred(out, self.w_output_weight, ctx, T)
             if part is not None:
@@ -165,10 +183,10 @@ class ShapedAttention(PagedAttention):
         linear(out, self.w_output_weight, residual, RESIDUAL if accumulate else STORE_F32, ctx, M=T)
         return None
 
-    def _finish(self, o, out, proj, ctx, vrot):
+    def _finish(self, o, out, proj, ctx, vrot, scale=1.0):
         """Turn back, gate, drop the padding past vdim and round once."""
         T, Hq, Hkv, Dk, Dv, Dp = ctx.n_tokens, self.Hq, self.Hkv, self.Dk, self.Dv, self.D
         off = Hq * Dk + Hkv * (Dk if self.value_from_key else Dk + Dv)
         gate = proj[:, off:off + Hq * Dv] if self.has_gate else None
         ops.attention_finish(o, T, ctx, vrot.cos_sin if vrot is not None else None, vrot.pairing if vrot is not None else 0,
-                             gate, out, Hq, Dv, Dp)
+                             gate, out, Hq, Dv, Dp, out_scale=scale)
