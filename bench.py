@@ -3,7 +3,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
                     [--model llama31-8b|llama32-3b|llama2-7b] [--dtype bf16|fp16|fp32]
-                    [--workload decode|serve|latent|hybrid|streams|delta] [--layers L] [--batch B] [--context S] [--trials N] [--size 2b|8b]
+                    [--workload decode|serve|latent|hybrid|streams|delta|decay] [--layers L] [--batch B] [--context S] [--trials N] [--size 2b|8b]
 
 Prints ONE JSON line.
 
@@ -47,6 +47,11 @@ pair of causal attention with a soft cap and a sink beside a matrix-memory recur
 values are its keys, and two gated delta rules with a decay per key channel; every layer with eight clamped experts
 plus two identity outputs, two per token, and a unit for every token) beside the closest of the other designs, a
 Vikupel of equal width, heads, layers and active feed-forward width.
+
+`--workload decay`: the same comparison for the Tikunex design (layers in turn: gated linear attention; windowed
+attention that keeps the first keys beside an RWKV-style recurrence; every layer with eight experts, three per token, and a
+per-layer token input; one pass of a loop around all layers) beside the closest of the other designs, a Pererax of equal
+width, heads, recurrent state, layers and feed-forward weights.
 
 Weights are random N(0, 0.02); token ids are uniform random from a seed.  No L2 flush is needed
 between steps: a step reads gigabytes of weights, far more than the 126 MB L2 holds.
@@ -193,8 +198,8 @@ def main():
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the model has (named in config)")
     ap.add_argument("--model", default="llama31-8b", choices=sorted(MODELS), help="layer sizes (random weights)")
     ap.add_argument("--dtype", default="bf16", choices=sorted(DTYPES), help="compute dtype; fp32 is the true 32-bit path")
-    ap.add_argument("--workload", default="decode", choices=["decode", "serve", "latent", "hybrid", "streams", "delta"])
-    ap.add_argument("--size", default="2b", choices=sorted(LATENT_SIZES), help="latent, hybrid, streams, delta: the layer sizes to compare at")
+    ap.add_argument("--workload", default="decode", choices=["decode", "serve", "latent", "hybrid", "streams", "delta", "decay"])
+    ap.add_argument("--size", default="2b", choices=sorted(LATENT_SIZES), help="latent, hybrid, streams, delta, decay: the layer sizes to compare at")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--context", type=int, default=None,
                     help="cached tokens per request of the headline point (default 8192 for llama31-8b, 4096 for "
@@ -221,6 +226,8 @@ def main():
         return latent(args, design="zavesun")
     if args.workload == "delta":
         return latent(args, design="pererax")
+    if args.workload == "decay":
+        return latent(args, design="tikunex")
     return decode(args)
 
 
@@ -618,10 +625,34 @@ def delta_configs(size, layers, vocab=32000, window=1024):
     return ours, hybrid_configs(size, layers, vocab, window)[0]
 
 
+# Tikunex at the same two widths: attention heads of 128 (a quarter as many KV heads), recurrent heads with a 128 x 128
+# memory each, eight experts, three per token: together as many feed-forward weights as the Pererax above, about as many active.
+DECAY_SIZES = {
+    "2b": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, memory_heads=16, rank=64, experts=8, top=3, expert_ff=1760, side=256),
+    "8b": dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=128, memory_heads=32, rank=64, experts=8, top=3, expert_ff=4480, side=256),
+}
+
+
+def decay_configs(size, layers, vocab=32000, window=1024):
+    """Layers in turn: gated linear attention, the pair; and the Pererax of equal size beside it."""
+    s = DECAY_SIZES[size]
+    gla = {"heads": s["memory_heads"], "dim": s["dim"], "vdim": s["vdim"], "tau": 16.0, "decay_rank": s["rank"]}
+    left = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["vdim"], "scale": s["dim"] ** -0.5,
+            "mask": {"size": window, "keep_first": 4}}
+    right = {"heads": s["memory_heads"], "dim": s["dim"], "decay_rank": s["rank"]}
+    mlp = {"kind": "moe", "expert": {"ff": s["expert_ff"]}, "router": {"experts": s["experts"], "top": s["top"]}}
+    kinds = [{"type": "gla", "mixer": gla},
+             {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 0.8, "right_scale": 0.6}}]
+    ours = {"architecture": "Tikunex", "vocab": vocab, "width": s["width"], "norm": {"eps": 1e-6}, "token_side": {"dim": s["side"]},
+            "loop": {"start": 0, "stop": layers, "times": 1}, "layers": [dict(kinds[i % 2], mlp=mlp) for i in range(layers)]}
+    return ours, delta_configs(size, layers, vocab, window)[0]
+
+
 # design -> (title, configs of the design and of the model beside it, sizes, window, what stands beside it)
 DESIGNS = {"ruperax": ("Ruperax", latent_configs, LATENT_SIZES, 4096, "llama"), "vikupel": ("Vikupel", hybrid_configs, HYBRID_SIZES, 1024, "llama"),
            "zavesun": ("Zavesun", stream_configs, STREAM_SIZES, 1024, "llama"),
-           "pererax": ("Pererax", delta_configs, DELTA_SIZES, 1024, "vikupel")}
+           "pererax": ("Pererax", delta_configs, DELTA_SIZES, 1024, "vikupel"),
+           "tikunex": ("Tikunex", decay_configs, DECAY_SIZES, 1024, "pererax")}
 
 
 def latent(args, design="ruperax"):

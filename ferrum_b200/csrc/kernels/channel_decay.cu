@@ -324,13 +324,19 @@ channel_decay_chain_kernel(const ChannelDecayArgs A) {
   float s = A.state[(long long)A.slots[r] * A.state_stride + off];
   const float* dec = A.seg_dec + ((size_t)first * A.H + h) * A.D + e / A.Dv;
   float* st = A.seg_state + (size_t)first * hs + off;
-  for (int i = 0; i < n; ++i) {
-    if (i < n - 1) {
-      const float own = st[(size_t)i * hs], p = dec[(size_t)i * A.H * A.D];
-      st[(size_t)i * hs] = s;
-      s = fmaf(p, s, own);
-    } else {
-      st[(size_t)i * hs] = s;
+  constexpr int BATCH = 8;                       // (the last segment has no contribution: nothing of it is read)
+  for (int i0 = 0; i0 < n; i0 += BATCH) {
+    float own[BATCH], p[BATCH];
+#pragma unroll
+    for (int i = 0; i < BATCH; ++i) {
+      const bool have = i0 + i < n - 1;
+      own[i] = have ? st[(size_t)(i0 + i) * hs] : 0.f;
+      p[i] = have ? dec[(size_t)(i0 + i) * A.H * A.D] : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < BATCH; ++i) {
+      if (i0 + i < n) st[(size_t)(i0 + i) * hs] = s;
+      s = fmaf(p[i], s, own[i]);
     }
   }
 }
@@ -390,13 +396,60 @@ FERRUM_API int ferrum_channel_decay(const float* q, int ldq, const float* k, int
 
 // ------------------------------------------------------------------ decays from a low-rank projection
 // z[t][n] = sum_r W2[n][r] act(low[t][r]) + bias[n]; out = exp(-exp(z)) (kind 0) or sigmoid(z)^(1/tau) (kind 1).
-// A block makes TM tokens x 64 channels, the inner size in steps of 32 through shared memory.
-template <typename T, int TM>
+__device__ __forceinline__ float cd_gate(float z, int kind, float inv_tau) {
+  return kind == 0 ? expf(-expf(z)) : expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau);
+}
+
+// A few tokens: a block of 8 tokens x 32 channels, a thread per pair; the tokens' low-rank rows wait in shared memory
+// (CD_GATE_ROWS elements at a time) and a channel's weights come straight from memory, eight at a time where they are aligned.
+constexpr int CD_GATE_ROWS = 128;
+template <typename T>
+__global__ void __launch_bounds__(256)
+channel_decay_gate_few_kernel(const float* __restrict__ low, int ldl, int rank, int act_tanh, const T* __restrict__ w2, const float* __restrict__ bias,
+                              int kind, float inv_tau, int n_tokens, int N, float* __restrict__ out, int ldo, int vec) {
+  __shared__ __align__(16) float sl[8][CD_GATE_ROWS];
+  const int tid = threadIdx.x, c = blockIdx.x * 32 + (tid & 31), i = tid >> 5;
+  const int t0 = blockIdx.y * 8;
+  const T* wr = w2 + (size_t)min(c, N - 1) * rank;
+  float acc = 0.f;
+  for (int k0 = 0; k0 < rank; k0 += CD_GATE_ROWS) {
+    const int n = min(CD_GATE_ROWS, rank - k0);
+    for (int idx = tid; idx < 8 * n; idx += 256) {
+      const int m = idx / n, k = idx % n;
+      const float v = t0 + m < n_tokens ? low[(size_t)(t0 + m) * ldl + k0 + k] : 0.f;
+      sl[m][k] = act_tanh ? tanhf(v) : v;
+    }
+    __syncthreads();
+    if (vec) {                       // (rank is a multiple of 8, and so is n)
+      for (int k = 0; k < n; k += 8) {
+        float wv[8];
+        if constexpr (sizeof(T) == 4) {
+          *reinterpret_cast<float4*>(&wv[0]) = *reinterpret_cast<const float4*>(wr + k0 + k);
+          *reinterpret_cast<float4*>(&wv[4]) = *reinterpret_cast<const float4*>(wr + k0 + k + 4);
+        } else {
+          const uint4 raw = *reinterpret_cast<const uint4*>(wr + k0 + k);
+          const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) wv[j] = to_f32<T>(e[j]);
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc = fmaf(sl[i][k + j], wv[j], acc);
+      }
+    } else {
+      for (int k = 0; k < n; ++k) acc = fmaf(sl[i][k], to_f32<T>(wr[k0 + k]), acc);
+    }
+    __syncthreads();
+  }
+  if (c < N && t0 + i < n_tokens) out[(size_t)(t0 + i) * ldo + c] = cd_gate(acc + bias[c], kind, inv_tau);
+}
+
+// Many tokens: a block makes 64 tokens x 64 channels, 4 x 4 a thread, the inner size in steps of 32 through shared memory.
+template <typename T>
 __global__ void __launch_bounds__(256)
 channel_decay_gate_kernel(const float* __restrict__ low, int ldl, int rank, int act_tanh, const T* __restrict__ w2, const float* __restrict__ bias,
                           int kind, float inv_tau, int n_tokens, int N, float* __restrict__ out, int ldo) {
-  constexpr int KC = 32, TN = 64, MT = TM / 16;
-  __shared__ float sl[KC][TM + 1], sw[KC][TN + 1];
+  constexpr int KC = 32, TN = 64, TM = 64, MT = 4;
+  __shared__ __align__(16) float sl[KC][TM + 4], sw[KC][TN + 4];
   const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
   const int n0 = blockIdx.x * TN, t0 = blockIdx.y * TM;
   float acc[MT][4];
@@ -417,11 +470,8 @@ channel_decay_gate_kernel(const float* __restrict__ low, int ldl, int rank, int 
     __syncthreads();
 #pragma unroll 8
     for (int k = 0; k < KC; ++k) {
-      float a[MT], b[4];
-#pragma unroll
-      for (int i = 0; i < MT; ++i) a[i] = sl[k][ty + 16 * i];
-#pragma unroll
-      for (int j = 0; j < 4; ++j) b[j] = sw[k][tx + 16 * j];
+      const float4 av = *reinterpret_cast<const float4*>(&sl[k][4 * ty]), bv = *reinterpret_cast<const float4*>(&sw[k][4 * tx]);
+      const float a[4] = {av.x, av.y, av.z, av.w}, b[4] = {bv.x, bv.y, bv.z, bv.w};
 #pragma unroll
       for (int i = 0; i < MT; ++i)
 #pragma unroll
@@ -431,15 +481,12 @@ channel_decay_gate_kernel(const float* __restrict__ low, int ldl, int rank, int 
   }
 #pragma unroll
   for (int i = 0; i < MT; ++i) {
-    const int t = t0 + ty + 16 * i;
+    const int t = t0 + 4 * ty + i;
     if (t >= n_tokens) continue;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      const int n = n0 + tx + 16 * j;
-      if (n >= N) continue;
-      const float z = acc[i][j] + bias[n];
-      const float r = kind == 0 ? expf(-expf(z)) : expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau);
-      out[(size_t)t * ldo + n] = r;
+      const int n = n0 + 4 * tx + j;
+      if (n < N) out[(size_t)t * ldo + n] = cd_gate(acc[i][j] + bias[n], kind, inv_tau);
     }
   }
 }
@@ -448,15 +495,16 @@ FERRUM_API int ferrum_channel_decay_gate(const float* low, int ldl, int rank, in
                                          float inv_tau, int n_tokens, int N, float* out, int ldo, cudaStream_t stream) {
   FERRUM_CHECK_ARG(rank > 0 && N > 0 && ldl >= rank && ldo >= N && (kind == 0 || kind == 1), "channel_decay_gate: bad sizes");
   if (n_tokens == 0) return 0;
-  const int tm = n_tokens <= 64 ? 16 : 64;
-  const dim3 grid((N + 63) / 64, (n_tokens + tm - 1) / tm);
+  const bool few = n_tokens <= 32;
+  const dim3 grid(few ? (N + 31) / 32 : (N + 63) / 64, few ? (n_tokens + 7) / 8 : (n_tokens + 63) / 64);
   FERRUM_CHECK_ARG(grid.y <= 65535, "channel_decay_gate: too many tokens");
-  if (tm == 16)
-    FERRUM_DISPATCH_DTYPE(dtype, T, (channel_decay_gate_kernel<T, 16><<<grid, 256, 0, stream>>>(low, ldl, rank, act_tanh, (const T*)w2, bias, kind,
-                                                                                               inv_tau, n_tokens, N, out, ldo)));
+  const int vec = rank % 8 == 0 && ((uintptr_t)w2 & 15) == 0;
+  if (few)
+    FERRUM_DISPATCH_DTYPE(dtype, T, (channel_decay_gate_few_kernel<T><<<grid, 256, 0, stream>>>(low, ldl, rank, act_tanh, (const T*)w2, bias, kind,
+                                                                                               inv_tau, n_tokens, N, out, ldo, vec)));
   else
-    FERRUM_DISPATCH_DTYPE(dtype, T, (channel_decay_gate_kernel<T, 64><<<grid, 256, 0, stream>>>(low, ldl, rank, act_tanh, (const T*)w2, bias, kind,
-                                                                                               inv_tau, n_tokens, N, out, ldo)));
+    FERRUM_DISPATCH_DTYPE(dtype, T, (channel_decay_gate_kernel<T><<<grid, 256, 0, stream>>>(low, ldl, rank, act_tanh, (const T*)w2, bias, kind,
+                                                                                           inv_tau, n_tokens, N, out, ldo)));
   FERRUM_CHECK_LAUNCH("channel_decay_gate");
   return 0;
 }

@@ -29,14 +29,19 @@ constexpr int MOE_MAX_TOP = 8;
 enum MoeScores : int { MOE_SIGMOID = 0, MOE_SOFTMAX = 1, MOE_CHOSEN_SOFTMAX = 2 };
 
 // ------------------------------------------------------------------ routing
-// logits [T][ldz] float32.  expert_of, rank_of [T*top] int32, weight_of [T*top] float32, counts [n_exp] (zero on entry).
-__global__ void __launch_bounds__(128)
-moe_route_kernel(const float* __restrict__ logits, int ldz, int n_tokens, int n_exp, int top, int score_kind, int renormalize,
-                 int* __restrict__ expert_of, int* __restrict__ rank_of, float* __restrict__ weight_of, int* __restrict__ counts,
-                 const float* __restrict__ correction, float weight_scale, int n_real, const float* __restrict__ bias) {
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int t = blockIdx.x * 4 + warp;
-  if (t >= n_tokens) return;
+// What a warp works out for token t: its `top` choices and their weights (every lane ends up with both).
+struct MoeRouter {
+  const float* logits;       // [T][ldz]
+  int ldz, n_exp, top, score_kind, renormalize;
+  const float* correction;   // [n_exp] or null
+  float weight_scale;
+  const float* bias;         // [n_exp] or null
+};
+__device__ __forceinline__ void moe_choose(const MoeRouter& R, int t, int lane, int (&chosen_e)[MOE_MAX_TOP], float (&chosen_w)[MOE_MAX_TOP]) {
+  const float* const logits = R.logits;
+  const float* const bias = R.bias;
+  const float* const correction = R.correction;
+  const int ldz = R.ldz, n_exp = R.n_exp, top = R.top, score_kind = R.score_kind;
   constexpr int PER = MOE_MAX_EXPERTS / 32;
   float s[PER];
   float mx = -INFINITY;
@@ -69,8 +74,6 @@ moe_route_kernel(const float* __restrict__ logits, int ldz, int n_tokens, int n_
     const int e = lane + 32 * i;
     pick[i] = (correction != nullptr && e < n_exp) ? s[i] + correction[e] : s[i];
   }
-  float chosen_w[MOE_MAX_TOP];
-  int chosen_e[MOE_MAX_TOP];
   float total = 0.f;
   for (int j = 0; j < top; ++j) {
     float best = -INFINITY, best_s = 0.f;
@@ -111,14 +114,77 @@ moe_route_kernel(const float* __restrict__ logits, int ldz, int n_tokens, int n_
     }
     for (int j = 0; j < top; ++j) chosen_w[j] /= sum;
   }
+  for (int j = 0; j < top; ++j) {
+    if (chosen_e[j] >= n_exp) chosen_e[j] = 0;      // (all scores NaN: expert 0 with a NaN weight)
+    chosen_w[j] = (R.renormalize ? chosen_w[j] / total : chosen_w[j]) * R.weight_scale;
+  }
+}
+
+// expert_of, rank_of [T*top] int32, weight_of [T*top] float32, counts [n_exp] (zero on entry).
+__global__ void __launch_bounds__(128)
+moe_route_kernel(const MoeRouter R, int n_tokens, int* __restrict__ expert_of, int* __restrict__ rank_of, float* __restrict__ weight_of,
+                 int* __restrict__ counts, int n_real) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * 4 + warp;
+  if (t >= n_tokens) return;
+  float chosen_w[MOE_MAX_TOP];
+  int chosen_e[MOE_MAX_TOP];
+  moe_choose(R, t, lane, chosen_e, chosen_w);
   if (lane == 0) {
-    for (int j = 0; j < top; ++j) {
-      const int e = chosen_e[j] < n_exp ? chosen_e[j] : 0;      // (all scores NaN: expert 0 with a NaN weight)
-      expert_of[(size_t)t * top + j] = e;
-      weight_of[(size_t)t * top + j] = (renormalize ? chosen_w[j] / total : chosen_w[j]) * weight_scale;
-      rank_of[(size_t)t * top + j] = e < n_real ? atomicAdd(&counts[e], 1) : 0;      // (an identity expert keeps no rows)
+    for (int j = 0; j < R.top; ++j) {
+      const int e = chosen_e[j];
+      expert_of[(size_t)t * R.top + j] = e;
+      weight_of[(size_t)t * R.top + j] = chosen_w[j];
+      rank_of[(size_t)t * R.top + j] = e < n_real ? atomicAdd(&counts[e], 1) : 0;      // (an identity expert keeps no rows)
     }
   }
+}
+
+// A few tokens: one launch.  Every block works out all tokens' choices (a warp a token), counts its own pair's place in
+// the sorted buffer from them, and gathers the row; block 0 also writes the counters.
+constexpr int MOE_FEW_TOKENS = 16, MOE_FEW_PAIRS = 256;
+template <typename T>
+__global__ void __launch_bounds__(MOE_FEW_PAIRS)
+moe_route_few_kernel(const MoeRouter R, int n_tokens, int* __restrict__ expert_of, int* __restrict__ rank_of, float* __restrict__ weight_of,
+                     int* __restrict__ counts, int n_real, const T* __restrict__ x, int ldx, int E, int scale_input, T* __restrict__ xg,
+                     int* __restrict__ row_of) {
+  __shared__ int se[MOE_FEW_PAIRS];
+  __shared__ float sw[MOE_FEW_PAIRS];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, top = R.top, np = n_tokens * top;
+  for (int t = warp; t < n_tokens; t += MOE_FEW_PAIRS / 32) {
+    float chosen_w[MOE_MAX_TOP];
+    int chosen_e[MOE_MAX_TOP];
+    moe_choose(R, t, lane, chosen_e, chosen_w);
+    if (lane == 0) {
+      for (int j = 0; j < top; ++j) {
+        se[t * top + j] = chosen_e[j];
+        sw[t * top + j] = chosen_w[j];
+      }
+    }
+  }
+  __syncthreads();
+  const int pair = blockIdx.x, e = se[pair];
+  const int mine = tid < np ? se[tid] : n_real;
+  const int first = __syncthreads_count(mine < n_real && mine < e);
+  const int rank = __syncthreads_count(tid < pair && mine == e);
+  const int row = e < n_real ? first + rank : -1;
+  const float w = sw[pair];
+  if (tid == 0) {
+    expert_of[pair] = e;
+    rank_of[pair] = row < 0 ? 0 : rank;
+    weight_of[pair] = w;
+    row_of[pair] = row;
+  }
+  if (pair == 0 && tid < n_real) {
+    int n = 0;
+    for (int i = 0; i < np; ++i) n += se[i] == tid;
+    counts[tid] = n;
+  }
+  if (row < 0) return;
+  const float f = scale_input ? w : 1.f;
+  const T* src = x + (size_t)(pair / top) * ldx;
+  T* dst = xg + (size_t)row * E;
+  for (int i = tid; i < E; i += MOE_FEW_PAIRS) dst[i] = from_f32<T>(to_f32<T>(src[i]) * f);
 }
 
 // x [T][ldx] -> xg [row][E] at the pair's place; row_of[pair] = row (-1 for an identity expert, which has no row).
@@ -580,17 +646,85 @@ moe_combine_kernel(const float* __restrict__ rows, int ld, const int* __restrict
                    int top, int E, float* __restrict__ y, const T* __restrict__ x, int ldx, const float* __restrict__ add,
                    int ld_add, int accumulate, T* __restrict__ yc, int ldyc) {
   const int t = blockIdx.x;
-  for (int i = threadIdx.x; i < E; i += 256) {
+  int row[MOE_MAX_TOP];
+  float wt[MOE_MAX_TOP];
+#pragma unroll
+  for (int j = 0; j < MOE_MAX_TOP; ++j) {
+    row[j] = j < top ? row_of[(size_t)t * top + j] : -1;
+    wt[j] = j < top && weight_of != nullptr ? weight_of[(size_t)t * top + j] : 1.f;
+  }
+  const int per = (E + gridDim.y - 1) / gridDim.y, end = min(E, (int)(blockIdx.y + 1) * per);
+  for (int i = blockIdx.y * per + threadIdx.x; i < end; i += 256) {
     float s = 0.f;
-    for (int j = 0; j < top; ++j) {
-      const int r = row_of[(size_t)t * top + j];
-      const float v = r >= 0 ? rows[(size_t)r * ld + i] : (x != nullptr ? to_f32<T>(x[(size_t)t * ldx + i]) : 0.f);
-      s += weight_of != nullptr ? v * weight_of[(size_t)t * top + j] : v;
+#pragma unroll
+    for (int j = 0; j < MOE_MAX_TOP; ++j) {
+      if (j < top) {
+        const int r = row[j];
+        const float v = r >= 0 ? rows[(size_t)r * ld + i] : (x != nullptr ? to_f32<T>(x[(size_t)t * ldx + i]) : 0.f);
+        s += weight_of != nullptr ? v * wt[j] : v;
+      }
     }
     if (add != nullptr) s += add[(size_t)t * ld_add + i];
     if (accumulate) s = y[(size_t)t * E + i] + s;
     y[(size_t)t * E + i] = s;
     if (yc != nullptr) yc[(size_t)t * ldyc + i] = from_f32<T>(s);
+  }
+}
+
+// The same sums in four columns a thread, for rows on 16-byte borders.
+template <typename T>
+__global__ void __launch_bounds__(256)
+moe_combine_vec_kernel(const float* __restrict__ rows, int ld, const int* __restrict__ row_of, const float* __restrict__ weight_of,
+                       int top, int E, float* __restrict__ y, const T* __restrict__ x, int ldx, const float* __restrict__ add,
+                       int ld_add, int accumulate, T* __restrict__ yc, int ldyc) {
+  const int t = blockIdx.x, i = (blockIdx.y * 256 + threadIdx.x) * 4;
+  if (i >= E) return;
+  auto load16 = [](const T* p) {
+    if constexpr (sizeof(T) == 4) {
+      return *reinterpret_cast<const float4*>(p);
+    } else {
+      const uint2 raw = *reinterpret_cast<const uint2*>(p);
+      const T* e = reinterpret_cast<const T*>(&raw);
+      return make_float4(to_f32<T>(e[0]), to_f32<T>(e[1]), to_f32<T>(e[2]), to_f32<T>(e[3]));
+    }
+  };
+  float4 v[MOE_MAX_TOP];
+  float wt[MOE_MAX_TOP];
+#pragma unroll
+  for (int j = 0; j < MOE_MAX_TOP; ++j) {
+    if (j < top) {
+      const int r = row_of[(size_t)t * top + j];
+      wt[j] = weight_of != nullptr ? weight_of[(size_t)t * top + j] : 1.f;
+      v[j] = r >= 0 ? *reinterpret_cast<const float4*>(rows + (size_t)r * ld + i) : (x != nullptr ? load16(x + (size_t)t * ldx + i) : make_float4(0.f, 0.f, 0.f, 0.f));
+    }
+  }
+  float4 old = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (accumulate) old = *reinterpret_cast<const float4*>(y + (size_t)t * E + i);
+  float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int j = 0; j < MOE_MAX_TOP; ++j) {
+    if (j < top) {
+      s.x += weight_of != nullptr ? v[j].x * wt[j] : v[j].x;
+      s.y += weight_of != nullptr ? v[j].y * wt[j] : v[j].y;
+      s.z += weight_of != nullptr ? v[j].z * wt[j] : v[j].z;
+      s.w += weight_of != nullptr ? v[j].w * wt[j] : v[j].w;
+    }
+  }
+  if (add != nullptr) {
+    const float4 a = *reinterpret_cast<const float4*>(add + (size_t)t * ld_add + i);
+    s.x += a.x, s.y += a.y, s.z += a.z, s.w += a.w;
+  }
+  s.x += old.x, s.y += old.y, s.z += old.z, s.w += old.w;
+  *reinterpret_cast<float4*>(y + (size_t)t * E + i) = s;
+  if (yc != nullptr) {
+    if constexpr (sizeof(T) == 4) {
+      *reinterpret_cast<float4*>(yc + (size_t)t * ldyc + i) = s;
+    } else {
+      uint2 pk;
+      pk.x = pack2<T>(s.x, s.y);
+      pk.y = pack2<T>(s.z, s.w);
+      *reinterpret_cast<uint2*>(yc + (size_t)t * ldyc + i) = pk;
+    }
   }
 }
 
@@ -618,10 +752,16 @@ FERRUM_API int ferrum_moe_route(const float* logits, int ldz, int n_tokens, int 
   const int n_real = n_exp - n_identity;
   FERRUM_CHECK_ARG(ldz >= n_exp && ldx >= E && E > 0, "moe_route: rows are shorter than their contents");
   if (n_tokens == 0) return 0;
+  const MoeRouter R{logits, ldz, n_exp, top, score_kind, renormalize, correction, weight_scale, bias};
+  if (n_tokens <= MOE_FEW_TOKENS && n_tokens * top <= MOE_FEW_PAIRS) {
+    FERRUM_DISPATCH_DTYPE(dtype, T, (moe_route_few_kernel<T><<<n_tokens * top, MOE_FEW_PAIRS, 0, stream>>>(
+        R, n_tokens, expert_of, rank_of, weight_of, counts, n_real, (const T*)x, ldx, E, scale_input, (T*)xg, row_of)));
+    FERRUM_CHECK_LAUNCH("moe_route (few tokens)");
+    return 0;
+  }
   cudaError_t e = cudaMemsetAsync(counts, 0, sizeof(int) * n_real, stream);
   FERRUM_CHECK_ARG(e == cudaSuccess, "moe_route: cannot clear the counters: %s", cudaGetErrorString(e));
-  moe_route_kernel<<<(n_tokens + 3) / 4, 128, 0, stream>>>(logits, ldz, n_tokens, n_exp, top, score_kind, renormalize,
-                                                           expert_of, rank_of, weight_of, counts, correction, weight_scale, n_real, bias);
+  moe_route_kernel<<<(n_tokens + 3) / 4, 128, 0, stream>>>(R, n_tokens, expert_of, rank_of, weight_of, counts, n_real);
   FERRUM_CHECK_LAUNCH("moe_route");
   FERRUM_DISPATCH_DTYPE(dtype, T, (moe_gather_kernel<T><<<n_tokens * top, 128, 0, stream>>>(
       (const T*)x, ldx, E, n_real, top, expert_of, rank_of, weight_of, counts, scale_input, (T*)xg, row_of)));
@@ -689,7 +829,16 @@ FERRUM_API int ferrum_moe_combine(const float* rows, int ld, const int* row_of, 
   FERRUM_CHECK_ARG(top > 0 && E > 0 && ld >= E, "moe_combine: bad sizes");
   FERRUM_CHECK_ARG((x == nullptr || ldx >= E) && (add == nullptr || ld_add >= E) && (yc == nullptr || ldyc >= E), "moe_combine: a row is shorter than the width");
   if (n_tokens == 0) return 0;
-  FERRUM_DISPATCH_DTYPE(x_dtype, T, (moe_combine_kernel<T><<<n_tokens, 256, 0, stream>>>(rows, ld, row_of, weight_of, top, E, y,
+  FERRUM_CHECK_ARG(top <= MOE_MAX_TOP && E <= 1 << 24, "moe_combine: %d choices per token are more than %d", top, MOE_MAX_TOP);
+  auto al = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+  if (E % 4 == 0 && ld % 4 == 0 && (x == nullptr || ldx % 4 == 0) && (add == nullptr || ld_add % 4 == 0) && (yc == nullptr || ldyc % 4 == 0) &&
+      al(rows) && al(y) && al(x) && al(add) && al(yc)) {
+    FERRUM_DISPATCH_DTYPE(x_dtype, T, (moe_combine_vec_kernel<T><<<dim3(n_tokens, (E + 1023) / 1024), 256, 0, stream>>>(
+        rows, ld, row_of, weight_of, top, E, y, (const T*)x, ldx, add, ld_add, accumulate, (T*)yc, ldyc)));
+    FERRUM_CHECK_LAUNCH("moe_combine");
+    return 0;
+  }
+  FERRUM_DISPATCH_DTYPE(x_dtype, T, (moe_combine_kernel<T><<<dim3(n_tokens, n_tokens <= 64 ? (E + 511) / 512 : 1), 256, 0, stream>>>(rows, ld, row_of, weight_of, top, E, y,
                                                                                        (const T*)x, ldx, add, ld_add, accumulate, (T*)yc, ldyc)));
   FERRUM_CHECK_LAUNCH("moe_combine");
   return 0;

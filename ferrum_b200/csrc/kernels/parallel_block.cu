@@ -6,7 +6,8 @@
 // gated_table_rows: g[t][j] = gelu_tanh(s[t][j]) * table[token[t]][offset + j]   (the per-layer part of a
 //                   second embedding table, gated by a projection of the row), compute type out.
 // norm_scaled_add:  x <- x + mult * y / sqrt(mean(y^2) + eps) * w    (an RMS norm of the branch's result,
-//                   not of x).
+//                   not of x); where rows lie on 16-byte borders it may go on to the norm that follows,
+//                   out <- x / sqrt(mean(x^2) + eps2) * w2 in the compute type, without reading x again.
 // All arithmetic is float32; one block per token for the norm, with a fixed reduction tree.
 #include "common.cuh"
 #include "partials.cuh"
@@ -98,6 +99,75 @@ norm_scaled_add_kernel(float* __restrict__ x, const float* __restrict__ y, const
   }
 }
 
+// Rows of E = 4 * (pieces) elements, at most PB_PIECES pieces a thread, kept in registers from the read to the last store.
+constexpr int PB_PIECES = 4;
+template <typename T>
+__global__ void __launch_bounds__(1024)
+norm_scaled_add_vec_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ w, float mult, float eps,
+                           int E, const PartialLayout L, const float* __restrict__ w2, float eps2, T* __restrict__ out) {
+  pdl_launch();      // the product that follows may fetch its weights meanwhile
+  __shared__ float red[32];
+  __shared__ PartialTable tab;
+  if (L.ws != nullptr) build_partial_table(L, tab);
+  const int t = blockIdx.x, n4 = E >> 2;
+  float4 v[PB_PIECES], xo[PB_PIECES];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < PB_PIECES; ++k) {
+    const int i = threadIdx.x + k * blockDim.x;
+    v[k] = xo[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < n4) {
+      xo[k] = *reinterpret_cast<const float4*>(x + (size_t)t * E + 4 * i);
+      if (L.ws != nullptr) {
+        v[k] = make_float4(partial_sum(L, tab, t, 4 * i), partial_sum(L, tab, t, 4 * i + 1), partial_sum(L, tab, t, 4 * i + 2),
+                           partial_sum(L, tab, t, 4 * i + 3));
+      } else {
+        v[k] = *reinterpret_cast<const float4*>(y + (size_t)t * E + 4 * i);
+      }
+    }
+    ss = fmaf(v[k].x, v[k].x, ss);
+    ss = fmaf(v[k].y, v[k].y, ss);
+    ss = fmaf(v[k].z, v[k].z, ss);
+    ss = fmaf(v[k].w, v[k].w, ss);
+  }
+  ss = block_sum(ss, red);
+  const float r = 1.f / sqrtf(ss / (float)E + eps);
+  float s2 = 0.f;
+#pragma unroll
+  for (int k = 0; k < PB_PIECES; ++k) {
+    const int i = threadIdx.x + k * blockDim.x;
+    if (i >= n4) continue;
+    const float4 g = *reinterpret_cast<const float4*>(w + 4 * i);
+    xo[k].x = fmaf(mult, v[k].x * r * g.x, xo[k].x);
+    xo[k].y = fmaf(mult, v[k].y * r * g.y, xo[k].y);
+    xo[k].z = fmaf(mult, v[k].z * r * g.z, xo[k].z);
+    xo[k].w = fmaf(mult, v[k].w * r * g.w, xo[k].w);
+    *reinterpret_cast<float4*>(x + (size_t)t * E + 4 * i) = xo[k];
+    s2 = fmaf(xo[k].x, xo[k].x, s2);
+    s2 = fmaf(xo[k].y, xo[k].y, s2);
+    s2 = fmaf(xo[k].z, xo[k].z, s2);
+    s2 = fmaf(xo[k].w, xo[k].w, s2);
+  }
+  if (out == nullptr) return;
+  s2 = block_sum(s2, red);
+  const float r2 = 1.f / sqrtf(s2 / (float)E + eps2);
+#pragma unroll
+  for (int k = 0; k < PB_PIECES; ++k) {
+    const int i = threadIdx.x + k * blockDim.x;
+    if (i >= n4) continue;
+    const float4 g = *reinterpret_cast<const float4*>(w2 + 4 * i);
+    const float a = xo[k].x * r2 * g.x, b = xo[k].y * r2 * g.y, c = xo[k].z * r2 * g.z, d = xo[k].w * r2 * g.w;
+    if constexpr (sizeof(T) == 4) {
+      *reinterpret_cast<float4*>(out + (size_t)t * E + 4 * i) = make_float4(a, b, c, d);
+    } else {
+      uint2 pk;
+      pk.x = pack2<T>(a, b);
+      pk.y = pack2<T>(c, d);
+      *reinterpret_cast<uint2*>(out + (size_t)t * E + 4 * i) = pk;
+    }
+  }
+}
+
 static int pb_layout(const float* partials, const int* layout, int n_tokens, int width, PartialLayout* L) {
   *L = PartialLayout{nullptr, 0, 0, 0, 0};
   if (partials == nullptr) return 0;
@@ -148,14 +218,34 @@ constexpr int PB_MAX_ROW = 11264;      // floats of a row that the norm holds in
 
 FERRUM_API int ferrum_norm_scaled_add_max_width() { return PB_MAX_ROW; }
 
+static bool pb_vec(const float* x, const float* y, const float* w, int E) {
+  return E % 4 == 0 && E <= 4096 * PB_PIECES && (((uintptr_t)x | (uintptr_t)y | (uintptr_t)w) & 15) == 0;
+}
+// Whether norm_scaled_add can go on to a norm of the new rows (w2 and out as below).
+FERRUM_API int ferrum_norm_scaled_add_can_norm(const float* x, const float* y, const float* w, int E, const float* w2, const void* out) {
+  return pb_vec(x, y, w, E) && (((uintptr_t)w2 | (uintptr_t)out) & 15) == 0;
+}
+
+// out (may be null): [n_tokens][E] in the type `dtype`, the norm of the new rows with weight w2 and eps2.
 FERRUM_API int ferrum_norm_scaled_add(float* x, const float* y, const float* w, float mult, float eps, int n_tokens, int E,
-                                      const float* partials, const int* layout, cudaStream_t stream) {
+                                      const float* partials, const int* layout, const float* w2, float eps2, void* out, int dtype,
+                                      cudaStream_t stream) {
   FERRUM_CHECK_ARG(y != nullptr || partials != nullptr, "norm_scaled_add: no input");
   FERRUM_CHECK_ARG(E > 0 && (partials == nullptr || E <= PB_MAX_ROW), "norm_scaled_add: a row of %d from partials is wider than %d",
                    E, PB_MAX_ROW);
   if (n_tokens == 0) return 0;
   PartialLayout L;
   if (int r = pb_layout(partials, layout, n_tokens, E, &L)) return r;
+  if (pb_vec(x, y, w, E)) {
+    FERRUM_CHECK_ARG(out == nullptr || (w2 != nullptr && (((uintptr_t)w2 | (uintptr_t)out) & 15) == 0), "norm_scaled_add: the norm's operands are unaligned");
+    // a few rows: a piece a thread; many: four, so that several rows share an SM
+    const int n4 = E / 4, most = n_tokens <= 64 ? n4 : (n4 + PB_PIECES - 1) / PB_PIECES;
+    const int threads = min(1024, max((most + 31) / 32 * 32, (n4 + 32 * PB_PIECES - 1) / (32 * PB_PIECES) * 32));
+    FERRUM_DISPATCH_DTYPE(dtype, T, (norm_scaled_add_vec_kernel<T><<<n_tokens, threads, 0, stream>>>(x, y, w, mult, eps, E, L, w2, eps2, (T*)out)));
+    FERRUM_CHECK_LAUNCH("norm_scaled_add");
+    return 0;
+  }
+  FERRUM_CHECK_ARG(out == nullptr, "norm_scaled_add: rows that are not on 16-byte borders take no norm after the sum");
   const int hold = E <= PB_MAX_ROW;
   norm_scaled_add_kernel<<<n_tokens, 256, hold ? (size_t)E * 4 : 0, stream>>>(x, y, w, mult, eps, E, L, hold);
   FERRUM_CHECK_LAUNCH("norm_scaled_add");

@@ -21,11 +21,6 @@ post_norm_add_kernel(float* __restrict__ h, int E, const float* __restrict__ y, 
   __shared__ float red[32];
   const int t = blockIdx.x;
   float* hr = h + (size_t)t * E;
-  if (y == nullptr) {
-    if (xc != nullptr)
-      for (int i = threadIdx.x; i < E; i += PN_THREADS) xc[(size_t)t * ldx + i] = from_f32<TX>(hr[i]);
-    return;
-  }
   const float* yr = y + (size_t)t * ldy;
   float ss = 0.f;
   for (int i = threadIdx.x; i < E; i += PN_THREADS) ss = fmaf(yr[i], yr[i], ss);
@@ -37,6 +32,14 @@ post_norm_add_kernel(float* __restrict__ h, int E, const float* __restrict__ y, 
     hr[i] = v;
     if (xc != nullptr) xc[(size_t)t * ldx + i] = from_f32<TX>(v);
   }
+}
+
+// Rows in the compute type alone: a row is shared out between gridDim.y blocks.
+template <typename TX>
+__global__ void __launch_bounds__(PN_THREADS)
+copy_rows_kernel(const float* __restrict__ h, int E, TX* __restrict__ xc, int ldx) {
+  const int i = blockIdx.y * PN_THREADS + threadIdx.x;
+  if (i < E) xc[(size_t)blockIdx.x * ldx + i] = from_f32<TX>(h[(size_t)blockIdx.x * E + i]);
 }
 
 __global__ void __launch_bounds__(PN_THREADS)
@@ -81,12 +84,73 @@ head_gate_norm_kernel(const float* __restrict__ o, int ldo, const float* __restr
   }
 }
 
+// The same where everything lies on 16-byte borders and a head has at most 512 elements: a lane keeps its pieces of the
+// head in registers between the sum of squares and the store.
+constexpr int PN_HEAD_PIECES = 4;
+template <typename T>
+__global__ void __launch_bounds__(128)
+head_gate_norm_vec_kernel(const float* __restrict__ o, int ldo, const float* __restrict__ gate, int ldg, const float* __restrict__ w,
+                          int w_per_head, float eps, int n_tokens, int H, int Dv, T* __restrict__ out, int ldout, int gate_silu,
+                          float out_scale) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * 4 + warp;
+  if (item >= (long long)n_tokens * H) return;
+  const int t = (int)(item / H), h = (int)(item % H);
+  const float4* src = reinterpret_cast<const float4*>(o + (size_t)t * ldo + (size_t)h * Dv);
+  const float4* g = gate != nullptr ? reinterpret_cast<const float4*>(gate + (size_t)t * ldg + (size_t)h * Dv) : nullptr;
+  const float4* wr = reinterpret_cast<const float4*>(w + (w_per_head ? (size_t)h * Dv : 0));
+  T* dst = out + (size_t)t * ldout + (size_t)h * Dv;
+  const int n4 = Dv >> 2;
+  float4 v[PN_HEAD_PIECES], gv[PN_HEAD_PIECES];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < PN_HEAD_PIECES; ++k) {
+    const int i = lane + 32 * k;
+    v[k] = i < n4 ? src[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    gv[k] = (g != nullptr && i < n4) ? g[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    ss = fmaf(v[k].x, v[k].x, ss);
+    ss = fmaf(v[k].y, v[k].y, ss);
+    ss = fmaf(v[k].z, v[k].z, ss);
+    ss = fmaf(v[k].w, v[k].w, ss);
+  }
+  ss = warp_sum(ss);
+  const float r = 1.f / sqrtf(ss / (float)Dv + eps);
+#pragma unroll
+  for (int k = 0; k < PN_HEAD_PIECES; ++k) {
+    const int i = lane + 32 * k;
+    if (i >= n4) continue;
+    const float4 ww = wr[i];
+    float e[4] = {v[k].x * r * ww.x, v[k].y * r * ww.y, v[k].z * r * ww.z, v[k].w * r * ww.w};
+    const float z[4] = {gv[k].x, gv[k].y, gv[k].z, gv[k].w};
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      if (g != nullptr) e[j] *= (gate_silu ? z[j] : 1.f) / (1.f + expf(-z[j]));
+      e[j] *= out_scale;
+    }
+    if constexpr (sizeof(T) == 4) {
+      *reinterpret_cast<float4*>(dst + 4 * i) = make_float4(e[0], e[1], e[2], e[3]);
+    } else {
+      uint2 pk;
+      pk.x = pack2<T>(e[0], e[1]);
+      pk.y = pack2<T>(e[2], e[3]);
+      *reinterpret_cast<uint2*>(dst + 4 * i) = pk;
+    }
+  }
+}
+
 // h [T, E] float32 += ls * rms(y) * w; xc (may be null): the new rows in the type `x_dtype`.  y null: only the copy.
 FERRUM_API int ferrum_post_norm_add(float* h, int E, const float* y, int ldy, const float* w, const float* ls, float eps,
                                     void* xc, int ldx, int x_dtype, int n_tokens, cudaStream_t stream) {
   FERRUM_CHECK_ARG(E > 0 && n_tokens >= 0 && (y == nullptr || (ldy >= E && w != nullptr)) && (xc == nullptr || ldx >= E),
                    "post_norm_add: bad sizes");
   if (n_tokens == 0 || (y == nullptr && xc == nullptr)) return 0;
+  if (y == nullptr) {
+    const dim3 grid(n_tokens, (E + PN_THREADS - 1) / PN_THREADS);
+    FERRUM_CHECK_ARG(grid.y <= 65535, "post_norm_add: rows are too wide");
+    FERRUM_DISPATCH_DTYPE(x_dtype, T, (copy_rows_kernel<T><<<grid, PN_THREADS, 0, stream>>>(h, E, (T*)xc, ldx)));
+    FERRUM_CHECK_LAUNCH("copy_rows");
+    return 0;
+  }
   FERRUM_DISPATCH_DTYPE(x_dtype, T, (post_norm_add_kernel<T><<<n_tokens, PN_THREADS, 0, stream>>>(h, E, y, ldy, w, ls, eps, (T*)xc, ldx)));
   FERRUM_CHECK_LAUNCH("post_norm_add");
   return 0;
@@ -111,6 +175,14 @@ FERRUM_API int ferrum_head_gate_norm(const float* o, int ldo, const float* gate,
   if (n_tokens == 0) return 0;
   const long long blocks = ((long long)n_tokens * H + 3) / 4;
   FERRUM_CHECK_ARG(blocks < (1LL << 31), "head_gate_norm: too many rows");
+  const bool vec = Dv % 4 == 0 && Dv <= 128 * PN_HEAD_PIECES && ldo % 4 == 0 && ldout % 4 == 0 && (gate == nullptr || ldg % 4 == 0) &&
+                   (((uintptr_t)o | (uintptr_t)gate | (uintptr_t)w | (uintptr_t)out) & 15) == 0;
+  if (vec) {
+    FERRUM_DISPATCH_DTYPE(dtype, T, (head_gate_norm_vec_kernel<T><<<(unsigned)blocks, 128, 0, stream>>>(o, ldo, gate, ldg, w, w_per_head, eps,
+                                                                                                    n_tokens, H, Dv, (T*)out, ldout, gate_silu, out_scale)));
+    FERRUM_CHECK_LAUNCH("head_gate_norm");
+    return 0;
+  }
   FERRUM_DISPATCH_DTYPE(dtype, T, (head_gate_norm_kernel<T><<<(unsigned)blocks, 128, 0, stream>>>(o, ldo, gate, ldg, w, w_per_head, eps,
                                                                                               n_tokens, H, Dv, (T*)out, ldout, gate_silu, out_scale)));
   FERRUM_CHECK_LAUNCH("head_gate_norm");

@@ -160,6 +160,9 @@ class StepContext:
         # A block that keeps several residual streams leaves its sublayer's write to the kernel that reads
         # the streams next: (streams tensor, S, E, ops.StreamWrite) or None.
         self.pending_streams = None
+        # A branch whose normed result joins the residual rows leaves that sum to the norm that reads them next:
+        # (residual tensor, ops.PendingAdd) or None.
+        self.pending_add = None
         self.defer_residuals = True
         self.defer_swiglu = True
         self.h2d_bytes = 0            # bytes copied to the device by the last fill
@@ -249,6 +252,7 @@ class StepContext:
         self.step_cache = {}
         self.pending_residual = None
         self.pending_streams = None
+        self.pending_add = None
 
     def buffers_generation(self):
         """Changes whenever a buffer that kernels read may have moved (a captured graph is stale then)."""
@@ -281,6 +285,22 @@ class StepContext:
             from ..ops import lib as ops
             self.pending_streams = None
             ops.hyper_step(p[0], p[1], p[2], self.n_tokens, write=p[3], store=True)
+        p = self.pending_add
+        if p is not None:
+            from ..ops import lib as ops
+            self.pending_add = None
+            ops.norm_scaled_add(p[0], p[1].y, p[1].w, p[1].mult, p[1].eps, self.n_tokens, partials=p[1].partials)
+
+    def take_pending_add(self, h):
+        """For a norm about to read all rows of `h`: the branch it must add first, or None."""
+        p = self.pending_add
+        if p is None:
+            return None
+        if p[0].data_ptr() == h.data_ptr():
+            self.pending_add = None
+            return p[1]
+        self.flush_residual()
+        return None
 
     def take_pending_streams(self, X):
         """For a kernel about to read the streams `X`: the write it must apply first, or None."""
@@ -297,6 +317,7 @@ class StepContext:
         """Nobody reads the residual rows any more in this step."""
         self.pending_residual = None
         self.pending_streams = None
+        self.pending_add = None
 
     # ------------------------------------------------------------------ scratch
     def buf(self, name, shape, dtype):

@@ -256,6 +256,14 @@ class Partials:
         self._c = (c_int * 4)(*layout)
 
 
+class PendingAdd:
+    """A sum into the residual rows that nobody has made yet, x += mult * y / sqrt(mean(y^2) + eps) * w: y a float32 buffer,
+    or a deferred product (`partials`)."""
+
+    def __init__(self, y, w, mult, eps, partials=None):
+        self.y, self.w, self.mult, self.eps, self.partials = y, w, mult, eps, partials
+
+
 def rmsnorm(x, weight, out, eps, rows=None, n_rows=None, partials=None, groups=1):
     """out[r] = rmsnorm(x[rows[r] if rows else r]) * weight; x float32, out float32 or bfloat16.
     With `partials` (a deferred residual product) the rows of x first get the partials added,
@@ -338,6 +346,41 @@ def gemm_generic(x, w, out, epilogue, M=None):
     _check(lib().ferrum_gemm_generic(_ptr(x), _ptr(w), _ptr(out), dtype_code(x.dtype), c_int(M), c_int(N), c_int(K),
                                      c_int(x.stride(0)), c_int(w.stride(0)), c_int(out.stride(0)), c_int(epilogue),
                                      _stream()), "gemm_generic")
+
+
+def thin_linear_supported(x, w, M):
+    """Whether x[:M] @ w.T has so few output features that `thin_linear` is the kernel to take."""
+    if w.shape[0] > 512 or x.dtype not in SIXTEEN_BIT or x.dtype != w.dtype or not w.is_contiguous() or not _thin_products:
+        return False
+    return bool(lib().ferrum_thin_linear_supported(_ptr(x), c_int(x.stride(0)), _ptr(w), dtype_code(x.dtype), c_int(M), c_int(w.shape[0]),
+                                                   c_int(w.shape[1])))
+
+
+_thin_products = True
+
+
+def set_thin_products(on: bool):
+    """Tests and measurements: False sends products of few features to the tensor-core kernel again."""
+    global _thin_products
+    _thin_products = bool(on)
+
+
+def thin_linear(x, w, out, M, err, table=None, offset=0, token_ids=None):
+    """out[:M] = x[:M] @ w.T for few output features; out float32 or the compute type.  With `table` (compute type
+    [vocabulary, columns]) out receives gelu_tanh(product) * table[token_ids[t], offset + n] in the compute type."""
+    _need16(x, "x", 2); _need16(w, "w", 2, like=x); _need(out, None, "out", 2)
+    N, K = w.shape
+    kind = 0 if out.dtype == torch.float32 else 1
+    if table is not None:
+        _need(table, x.dtype, "table", 2); _need(token_ids, torch.int32, "token_ids", 1)
+        kind = 2
+    if x.shape[1] != K or out.shape[1] < N or min(x.shape[0], out.shape[0]) < M or (kind and out.dtype != x.dtype):
+        raise KernelError("thin_linear: shapes do not agree")
+    _gemm_work(x, w, out, M, N, K)
+    _check(lib().ferrum_thin_linear(_ptr(x), c_int(x.stride(0)), _ptr(w), dtype_code(x.dtype), c_int(M), c_int(N), c_int(K), c_int(kind),
+                                    _ptr(out), c_int(out.stride(0)), _ptr(table), c_int(table.stride(0) if table is not None else 0),
+                                    c_int(table.shape[0] if table is not None else 0), c_int(offset), _ptr(token_ids), _ptr(err),
+                                    _stream()), "thin_linear")
 
 
 def gemm_tc_supported(x, w):
@@ -911,8 +954,19 @@ def norm_scaled_add_max_width():
     return int(lib().ferrum_norm_scaled_add_max_width())
 
 
-def norm_scaled_add(x, y, w, mult, eps, n_tokens, partials=None):
-    """x[:n] += mult * y / sqrt(mean(y^2) + eps) * w, all float32; y a buffer or a deferred product (`partials`)."""
+def norm_scaled_add_can_norm(x, y, w, w2, out):
+    """Whether `norm_scaled_add(..., norm=(w2, eps, out))` is possible for these tensors (y None: partials)."""
+    return bool(lib().ferrum_norm_scaled_add_can_norm(_ptr(x), _ptr(y), _ptr(w), c_int(x.shape[1]), _ptr(w2), _ptr(out)))
+
+
+def norm_scaled_add(x, y, w, mult, eps, n_tokens, partials=None, norm=None):
+    """x[:n] += mult * y / sqrt(mean(y^2) + eps) * w, all float32; y a buffer or a deferred product (`partials`).
+    norm=(w2, eps2, out): out[:n] = x / sqrt(mean(x^2) + eps2) * w2 of the new rows, in out's type."""
+    w2, eps2, out = norm if norm is not None else (None, 0.0, None)
+    if out is not None:
+        _need(w2, torch.float32, "w2", 1); _need(out, None, "out", 2)
+        if w2.shape[0] != x.shape[1] or out.shape[1] != x.shape[1] or not out.is_contiguous() or out.shape[0] < n_tokens:
+            raise KernelError("norm_scaled_add: shapes do not agree")
     _need(x, torch.float32, "x", 2); _need(w, torch.float32, "w", 1)
     E = x.shape[1]
     if partials is None:
@@ -921,9 +975,10 @@ def norm_scaled_add(x, y, w, mult, eps, n_tokens, partials=None):
             raise KernelError("norm_scaled_add: shapes do not agree")
     if w.shape[0] != E or not x.is_contiguous():
         raise KernelError("norm_scaled_add: shapes do not agree")
-    _bytes_work((x, 2 * n_tokens), (x, n_tokens))
+    _bytes_work((x, 2 * n_tokens), (x, n_tokens), (out, n_tokens))
     _check(lib().ferrum_norm_scaled_add(_ptr(x), _ptr(y if partials is None else None), _ptr(w), c_float(mult), c_float(eps),
-                                        c_int(n_tokens), c_int(E), *_partials_args(partials), _stream()), "norm_scaled_add")
+                                        c_int(n_tokens), c_int(E), *_partials_args(partials), _ptr(w2), c_float(eps2), _ptr(out),
+                                        dtype_code(out.dtype if out is not None else torch.float32), _stream()), "norm_scaled_add")
 
 
 # ----------------------------------------------------------------------------- several residual streams
@@ -1013,7 +1068,7 @@ def moe_route(logits, n_tokens, n_exp, top, x, scale_input, expert_of, rank_of, 
                                   dtype_code(x.dtype), c_int(1 if scale_input else 0), _ptr(expert_of), _ptr(rank_of),
                                   _ptr(weight_of), _ptr(counts), _ptr(xg), _ptr(row_of), _ptr(correction), c_float(weight_scale),
                                   c_int(n_identity), _ptr(bias), _stream()), "moe_route")
-    launches += 1          # (the entry point launches the routing and the gather)
+    launches += 0 if n_tokens <= 16 and n_tokens * top <= 256 else 1          # (with many tokens: the routing and the gather)
 
 
 _moe_tcgen05 = True

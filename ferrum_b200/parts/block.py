@@ -52,7 +52,7 @@ class PreNormBlock(Part):
             ctx.flush_residual()
             if not copied:
                 ops.post_norm_add(h, ctx.n_tokens, xc=rows)
-            self.side.forward(h, rows, ctx, 1.0)
+            self.side.forward(h, rows, ctx, 1.0, defer=True)
 
 
 class RestartInput(Part):
@@ -279,21 +279,28 @@ class TokenSideInput(Part):
         return {"gate.weight": ParamSpec((self.dim, self.width)), "proj.weight": ParamSpec((self.width, self.dim)),
                 "norm.weight": ParamSpec((self.width,), kind="vector", init="ones_normal")}
 
-    def forward(self, h, x_in, ctx, mult):
-        """h: the float32 residual rows (updated in place); x_in: the same rows in the compute type."""
+    def forward(self, h, x_in, ctx, mult, defer=False):
+        """h: the float32 residual rows (updated in place; with defer=True their sum with the branch stays pending in `ctx`
+        for the norm that reads them next, see StepContext.pending_add); x_in: the same rows in the compute type."""
         T, cap = ctx.n_tokens, ctx.token_capacity
-        few = T <= OVERLAP_MAX_TOKENS       # a few tokens: both products stay in partials, summed by the kernels that follow
-        s = ctx.buf("side_s", (cap, self.dim), torch.float32)
-        part = linear_deferred(x_in, self.w_gate_weight, ctx, T) if few else None
-        if part is None:
-            linear(x_in, self.w_gate_weight, s, STORE_F32, ctx, M=T)
+        few = T <= OVERLAP_MAX_TOKENS       # a few tokens: the products stay in partials, summed by the kernels that follow
         g = ctx.buf("side_g", (cap, self.dim), self.dtype)
-        ops.gated_table_rows(s, self.table.w_weight, ctx.token_ids, self.offset, self.dim, g, T, ctx.err, partials=part)
+        if ops.thin_linear_supported(x_in, self.w_gate_weight, T):
+            ctx.flush_residual()
+            ops.thin_linear(x_in, self.w_gate_weight, g, T, ctx.err, table=self.table.w_weight, offset=self.offset, token_ids=ctx.token_ids)
+        else:
+            s = ctx.buf("side_s", (cap, self.dim), torch.float32)
+            part = linear_deferred(x_in, self.w_gate_weight, ctx, T) if few else None
+            if part is None:
+                linear(x_in, self.w_gate_weight, s, STORE_F32, ctx, M=T)
+            ops.gated_table_rows(s, self.table.w_weight, ctx.token_ids, self.offset, self.dim, g, T, ctx.err, partials=part)
         y = ctx.buf("side_y", (cap, self.width), torch.float32)
         part = linear_deferred(g, self.w_proj_weight, ctx, T) if few and self.width <= ops.norm_scaled_add_max_width() else None
         if part is None:
             linear(g, self.w_proj_weight, y, STORE_F32, ctx, M=T)
-        ops.norm_scaled_add(h, y, self.w_norm_weight, mult, self.eps, T, partials=part)
+        ctx.pending_add = (h, ops.PendingAdd(y, self.w_norm_weight, mult, self.eps, part))
+        if not defer:
+            ctx.flush_residual()
 
 
 class ParallelBlock(Part):
@@ -357,7 +364,7 @@ class ParallelBlock(Part):
             xc = ctx.buf("par_xc", (cap, E), self.side.dtype)
         ops.scaled_sum(h, y1, y2, self.mult, T, xc, p1=p1, p2=p2)
         if self.side is not None:
-            self.side.forward(h, xc if xc is not None else h, ctx, self.mult)
+            self.side.forward(h, xc if xc is not None else h, ctx, self.mult, defer=True)
 
 
 def _stream_init(kind):

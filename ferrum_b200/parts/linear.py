@@ -1,4 +1,5 @@
-"""y = x W^T for the parts: picks the tensor-core kernel when the operands allow it.
+"""y = x W^T for the parts: picks the tensor-core kernel when the operands allow it (and the thin product's kernel
+when there are too few output features to make tiles of).
 
 The weight keeps the file's layout [out_features, in_features] with the input dimension
 contiguous (the reference's GEMV layout, crates/model/src/weights.rs:124-140), which is the
@@ -18,7 +19,7 @@ def linear_deferred(x, w, ctx, M, N=None, dual_offset=0):
     """The product as float32 partials for the next kernel to sum (`ops.Partials`), or None
     when the shape or the operands do not allow it.  The partials live in the step's product
     workspace: they must be consumed before the next tensor-core product runs."""
-    if M == 0 or not ops.gemm_tc_supported(x, w):
+    if M == 0 or not ops.gemm_tc_supported(x, w) or (N is None and not dual_offset and ops.thin_linear_supported(x, w, M)):
         return None
     N = (w.shape[0] - dual_offset) if N is None else N
     K = w.shape[1]
@@ -41,7 +42,9 @@ def linear(x, w, out, mode, ctx, M=None):
             ctx.pending_residual = (out, part)
             return
     ctx.flush_residual()
-    if ops.gemm_tc_supported(x, w):
+    if mode != RESIDUAL and ops.thin_linear_supported(x, w, M):
+        ops.thin_linear(x, w, out, M, ctx.err)
+    elif ops.gemm_tc_supported(x, w):
         N, K = w.shape
         ws, cnt = ctx.gemm_scratch(M, N, K, False)
         ops.gemm_tc(x, w, out, _TC[mode], ctx.err, ws, cnt, M=M)

@@ -34,5 +34,14 @@ class RMSNorm(Norm):
             ctx.flush_residual()
             ops.rmsnorm(h, self.w_weight, out, self.eps, rows=rows, n_rows=n, groups=self.groups)
             return out
+        if rows is None and ctx.pending_add is not None:
+            p = ctx.take_pending_add(h)
+            if p is not None:
+                if ops.norm_scaled_add_can_norm(h, p.y if p.partials is None else None, p.w, self.w_weight, out):
+                    ops.norm_scaled_add(h, p.y, p.w, p.mult, p.eps, n, partials=p.partials, norm=(self.w_weight, self.eps, out))
+                    return out
+                ops.norm_scaled_add(h, p.y, p.w, p.mult, p.eps, n, partials=p.partials)
+        elif ctx.pending_add is not None:
+            ctx.flush_residual()
         ops.rmsnorm(h, self.w_weight, out, self.eps, rows=rows, n_rows=n, partials=ctx.take_pending_residual(h))
         return out

@@ -12,6 +12,7 @@ peaks.  This is the small case that `ncu` captures are taken on.
     python kernel_bench.py attn_decode|attn_prefill --exact [--window W] [--penalty]   (float32 weights and sums on 16-bit storage)
     python kernel_bench.py ssm --tokens 2048 [--batch 1] [--hq 64] [--head-dim 64] [--state 128]   (the state-space mixer's kernels)
     python kernel_bench.py delta|memory --tokens 2048 [--batch 1] [--hq 16] [--head-dim 128]   (the walks of the gated delta rule and of the matrix memory)
+    python kernel_bench.py cdecay --tokens 2048 [--batch 1] [--hq 16] [--head-dim 128] [--bonus] [--segment L]   (the walk with a decay per key channel)
     python kernel_bench.py moe --tokens 4096 --n 2816 --k 2048 [--experts 8] [--epilogue store|swiglu] [--mma-sync] [--cuda-cores]   (grouped product of a routed feed-forward)
     python kernel_bench.py streams --tokens 2048 --k 2048 [--streams 4]   (write, read and norm over the residual streams)
     python kernel_bench.py rmsnorm|rope --tokens 8
@@ -39,7 +40,9 @@ sys.path.insert(0, ROOT)
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("kernel", choices=["attn_decode", "attn_prefill", "latent_decode", "latent_prefill", "head_linear", "gemm", "moe", "streams", "rmsnorm",
-                                       "rope", "ssm", "delta", "memory", "step", "timeline"])
+                                       "rope", "ssm", "delta", "memory", "cdecay", "step", "timeline"])
+    ap.add_argument("--bonus", action="store_true", help="cdecay: the read-out before the write, with a bonus for the current token")
+    ap.add_argument("--segment", type=int, default=-1, help="cdecay: tokens per segment (0: one piece; -1: the library's choice)")
     ap.add_argument("--kv-rank", type=int, default=512, help="latent_*: elements of the cached latent (the values)")
     ap.add_argument("--rot-dim", type=int, default=64, help="latent_*: rotated key elements behind the latent")
     ap.add_argument("--window", type=int, default=0, help="latent_*: keys a query looks back over (0: all)")
@@ -175,6 +178,22 @@ def main():
             gates = torch.empty(T, 2 * H, device=dev)
             runs = [lambda st=st: ops.matrix_memory(proj, offs, bi, bf, 12.0, T, ctx, H, Dk, Dk, st, gates, o) for st in states]
             work = {"bytes": 4 * (T * (4 * H * Dk + 2 * H) + 2 * R * H * Dk * Dk), "flops": 4.0 * T * H * Dk * Dk, "bound": "ffma"}
+    elif args.kernel == "cdecay":
+        # --batch requests of --tokens tokens each; --hq heads with keys and values of --head-dim elements
+        H, Dk, R, n = Hq, D, args.batch, args.tokens
+        T = R * n
+        ctx = StepContext(dev, max(16, T), R, [])
+        ctx.fill([StepEntry(r, 0, [1] * n) for r in range(R)], [])
+        f = lambda *shape: torch.randn(*shape, device=dev, generator=gen) * 0.2
+        proj, o = f(T, 3 * H * Dk), torch.empty(T, H * Dk, device=dev)
+        dec = torch.rand(T, H * Dk, device=dev, generator=gen)
+        bonus = f(H, Dk) if args.bonus else None
+        states = [torch.zeros(R, H * Dk * Dk, device=dev) for _ in range(args.layers)]
+        cut = None if args.segment < 0 else (args.segment, R * -(-n // args.segment) if args.segment else 0)
+        w = H * Dk
+        runs = [lambda st=st: ops.channel_decay(proj[:, :w], proj[:, w:2 * w], proj[:, 2 * w:], dec, T, ctx, H, Dk, Dk, st, o, bonus=bonus,
+                                                segments=cut) for st in states]
+        work = {"bytes": 4 * (T * 5 * w + 2 * R * w * Dk), "flops": 5.0 * T * w * Dk, "bound": "hbm" if n == 1 else "ffma"}
     elif args.kernel in ("latent_decode", "latent_prefill"):
         # attention over cached rows of kv_rank + rot_dim elements, --hq heads sharing them
         decode = args.kernel == "latent_decode"

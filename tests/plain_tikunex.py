@@ -138,11 +138,12 @@ def rwkv(x, w, pre, m, eps, round_to=None):
     """Returns the gated heads side by side (no output matrix)."""
     T = x.shape[0]
     H, D = m["heads"], m["dim"]
+    x = rnd(x, round_to)             # (what the token before leaves behind is its rounded row)
     mix = {s: shifted_mix(x, w[pre + "mu." + s]) for s in "rkvgw"}
     r, k, v = (matmul(mix[s], w[pre + s], round_to).reshape(T, H, D) for s in "rkv")
     gate = silu(matmul(mix["g"], w[pre + "g"], round_to))
-    low = torch.tanh(matmul(mix["w"], w[pre + "w1"], round_to))
-    dec = torch.exp(-torch.exp(matmul(low, w[pre + "w2"], round_to) + w[pre + "w0"])).reshape(T, H, D)
+    low = torch.tanh(matmul(mix["w"], w[pre + "w1"], round_to))          # (stays 32-bit on its way into the decay)
+    dec = torch.exp(-torch.exp(low @ rnd(w[pre + "w2"], round_to).T + w[pre + "w0"])).reshape(T, H, D)
     o = rms(rwkv_walk(r, k, v, dec, w[pre + "u"]), eps).reshape(T, H * D)
     return o * w[pre + "norm"] * gate
 
@@ -172,7 +173,7 @@ def gla(x, w, pre, m, eps, round_to=None):
     q = matmul(x, w[pre + "q"], round_to).reshape(T, H, D) * D ** -0.5
     k = matmul(x, w[pre + "k"], round_to).reshape(T, H, D)
     v = matmul(x, w[pre + "v"], round_to).reshape(T, H, Dv)
-    z = matmul(matmul(x, w[pre + "a1"], round_to), w[pre + "a2"], round_to) + w[pre + "a2.b"]
+    z = matmul(x, w[pre + "a1"], round_to) @ rnd(w[pre + "a2"], round_to).T + w[pre + "a2.b"]
     alpha = (torch.sigmoid(z) ** (1.0 / m["tau"])).reshape(T, H, D)
     o = (rms(gla_walk(q, k, v, alpha), eps) * w[pre + "norm"]).reshape(T, H * Dv)
     return matmul(o * silu(matmul(x, w[pre + "g"], round_to)), w[pre + "o"], round_to)
