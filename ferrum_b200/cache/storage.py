@@ -5,7 +5,8 @@ same (kv heads, head size, window, parts, kept first positions) form a group; ea
 the group's pool, a run with `cache_of` shares the plane of the run it names (it may look back
 over another window: the plane then keeps what the widest of its readers needs).  Runs whose
 mixers (or blocks) keep a fixed-size state get a state array [max_requests, ...] indexed by slot
-id; a state always belongs to one run, also when the run reads another run's pages.
+id; a state always belongs to one run, also when the run reads another run's pages, or to the
+model's embedding (`embedding_need`), which may look back at a request's tokens.
 
 `CacheStorage` allocates one pool per group, [planes, pages, parts (K, V; or one), kv heads,
 page_size, head size] in the compute dtype, the state arrays, and the native `CacheManager` that owns
@@ -85,6 +86,12 @@ class CacheLayout:
             else:
                 self.run_state.append(None)
 
+        need = model.embedding_need() if hasattr(model, "embedding_need") else None
+        self.embedding_state: Optional[int] = None
+        if need is not None and need.state is not None:
+            self.embedding_state = len(self.state_needs)
+            self.state_needs.append(need.state)
+
     def bytes_per_token(self, dtype) -> int:
         size = torch.empty((), dtype=dtype).element_size()
         return sum(parts * h * d * planes * size for (h, d, _, parts), planes in zip(self.group_keys, self.group_planes))
@@ -137,6 +144,12 @@ class CacheStorage:
 
     def layer_cache(self, k) -> LayerCache:
         return self._views[k]
+
+    @property
+    def embedding_state(self) -> Optional[torch.Tensor]:
+        """The embedding's state rows [max_requests, ...], or None."""
+        i = self.layout.embedding_state
+        return self.states[i] if i is not None else None
 
     @property
     def n_groups(self):

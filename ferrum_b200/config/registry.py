@@ -95,3 +95,5 @@ def _ensure_builtin():
         from ..models import pererax  # noqa: F401
     if "Tikunex" not in _REGISTRY:
         from ..models import tikunex  # noqa: F401
+    if "Lelutar" not in _REGISTRY:
+        from ..models import lelutar  # noqa: F401

@@ -14,9 +14,13 @@
 // portions: 12 warps on one key stage).  Key stages arrive by cp.async one stage
 // ahead.  Single tokens may cut their key range at multiples of 128 absolute positions among CTAs
 // (partials folded by attention_latent_combine, the same as the CUDA-core kernel's).
+// `wide` keeps the softmax weights to float32 precision on their way into the matrix unit: a weight goes in as its
+// rounding to the 16-bit type and the rounding of what that leaves out, two operand tiles whose products meet in the
+// same float32 accumulator (relative error of a weight 2^-17 for bfloat16 instead of 2^-9).
 // Needs Dk % 16 == 0, Dv % 32 == 0, Dv <= 512 and 16-byte aligned rows; the CUDA-core kernel takes
 // everything else and float32.
 #include "common.cuh"
+#include "softmax_sink.cuh"
 
 #include <type_traits>
 
@@ -56,30 +60,30 @@ __device__ __forceinline__ void lm_mma(float (&d)[4], const uint32_t (&a)[4], ui
 struct LmSmem {
   int DKP, off_k, off_s, off_row, bytes;     // offsets in bytes
 };
-inline LmSmem lm_smem(int Dk, int NRT, int TK) {
+inline LmSmem lm_smem(int Dk, int NRT, int TK, int wide) {
   LmSmem s;
   s.DKP = Dk + 8;                                    // (rows 16 bytes apart modulo 128: ldmatrix reads eight rows without bank conflicts)
   s.off_k = NRT * 16 * s.DKP * 2;
-  s.off_s = s.off_k + 2 * TK * s.DKP * 2;                // per row tile: 64 + 64 floats (maxima, sums), then its weights tile
-  s.off_row = s.off_s + NRT * (128 * 4 + 16 * (TK + 8) * 2);
+  s.off_s = s.off_k + 2 * TK * s.DKP * 2;                // per row tile: 64 + 64 floats (maxima, sums), then its weights tile(s)
+  s.off_row = s.off_s + NRT * (128 * 4 + (wide ? 2 : 1) * 16 * (TK + 8) * 2);
   s.bytes = s.off_row + 2 * TK * 8;
   return s;
 }
 
 // NV: n-tiles of 8 value columns per warp (Dv / 32 <= NV).  NRT: row tiles per CTA.
-template <typename T, int NV, int NRT, int TK>
+template <typename T, int NV, int NRT, int TK, bool WIDE>
 __global__ void __launch_bounds__(128 * NRT)
 attention_latent_mma_kernel(const T* __restrict__ q, int ldq, T* __restrict__ out, int ldo, const float* __restrict__ gate,
                             const int* __restrict__ positions, const int* __restrict__ q_start, int n_reqs,
                             const int* __restrict__ block_table, int table_width, const T* __restrict__ plane,
                             long long page_stride, int page_size, int H, int HB, int Dk, int Dv, float scale, int window,
                             int* __restrict__ err, int DKP, int off_k, int off_s, int off_row, float* __restrict__ part,
-                            int split_slots) {
+                            int split_slots, const float* __restrict__ sink) {
   extern __shared__ __align__(16) unsigned char lm_sm[];
   T* const sQ = reinterpret_cast<T*>(lm_sm);
   T* const sK = reinterpret_cast<T*>(lm_sm + off_k);
   float* const sS = reinterpret_cast<float*>(lm_sm + off_s);                        // [NRT][64] maxima, [NRT][64] sums
-  T* const sP = reinterpret_cast<T*>(lm_sm + off_s + NRT * 128 * 4);                // [NRT * 16][LM_PS]
+  T* const sP = reinterpret_cast<T*>(lm_sm + off_s + NRT * 128 * 4);                // [NRT * 16][LM_PS] (WIDE: and the remainders behind)
   long long* const sRow = reinterpret_cast<long long*>(lm_sm + off_row);
   __shared__ int chunk_req, chunk_t0, chunk_nt;
   constexpr int THREADS = 128 * NRT;
@@ -276,7 +280,7 @@ attention_latent_mma_kernel(const T* __restrict__ q, int ldq, T* __restrict__ ou
       }
       __syncthreads();               // the four warps' maxima are there
       float corr[2];
-      uint32_t pw[2][2];
+      uint32_t pw[2][2], pr[2][2];
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         const int r = (lane >> 2) + 8 * j;
@@ -296,6 +300,12 @@ attention_latent_mma_kernel(const T* __restrict__ q, int ldq, T* __restrict__ ou
         m[j] = m_new;
         pw[j][0] = pack2<T>(sv[j][0], sv[j][1]);
         pw[j][1] = pack2<T>(sv[j][2], sv[j][3]);
+        if constexpr (WIDE) {
+          const T* hi0 = reinterpret_cast<const T*>(&pw[j][0]);
+          const T* hi1 = reinterpret_cast<const T*>(&pw[j][1]);
+          pr[j][0] = pack2<T>(sv[j][0] - to_f32<T>(hi0[0]), sv[j][1] - to_f32<T>(hi0[1]));
+          pr[j][1] = pack2<T>(sv[j][2] - to_f32<T>(hi1[0]), sv[j][3] - to_f32<T>(hi1[1]));
+        }
       }
       // the weights, rounded to the storage type, into the row tile's [16][TK] operand tile
       T* const sPt = sP + rt * 16 * LM_PS;
@@ -306,6 +316,15 @@ attention_latent_mma_kernel(const T* __restrict__ q, int ldq, T* __restrict__ ou
         *reinterpret_cast<uint32_t*>(&sPt[r0 * LM_PS + cc + 8]) = pw[0][1];
         *reinterpret_cast<uint32_t*>(&sPt[(r0 + 8) * LM_PS + cc + 8]) = pw[1][1];
       }
+      if constexpr (WIDE) {
+        T* const sPr = sPt + NRT * 16 * LM_PS;
+        *reinterpret_cast<uint32_t*>(&sPr[r0 * LM_PS + cc]) = pr[0][0];
+        *reinterpret_cast<uint32_t*>(&sPr[(r0 + 8) * LM_PS + cc]) = pr[1][0];
+        if constexpr (KW == 16) {
+          *reinterpret_cast<uint32_t*>(&sPr[r0 * LM_PS + cc + 8]) = pr[0][1];
+          *reinterpret_cast<uint32_t*>(&sPr[(r0 + 8) * LM_PS + cc + 8]) = pr[1][1];
+        }
+      }
 #pragma unroll
       for (int j = 0; j < NV; ++j) {
         acc[j][0] *= corr[0];
@@ -315,7 +334,10 @@ attention_latent_mma_kernel(const T* __restrict__ q, int ldq, T* __restrict__ ou
       }
     }
     __syncthreads();                 // the row tile's weights are complete
-    uint32_t pa[TK / 16][4];
+    uint32_t pa[TK / 16][4], pb[WIDE ? TK / 16 : 1][4];
+#pragma unroll
+    for (int kk = 0; kk < (WIDE ? TK / 16 : 0); ++kk)
+      lm_ldmatrix_x4(pb[kk], sP + (size_t)(NRT * 16 + rt * 16 + (lane & 15)) * LM_PS + kk * 16 + (lane >> 4) * 8);
 #pragma unroll
     for (int kk = 0; kk < TK / 16; ++kk)
       lm_ldmatrix_x4(pa[kk], sP + (size_t)(rt * 16 + (lane & 15)) * LM_PS + kk * 16 + (lane >> 4) * 8);
@@ -330,6 +352,10 @@ attention_latent_mma_kernel(const T* __restrict__ q, int ldq, T* __restrict__ ou
           lm_ldmatrix_x4_trans(bv, vr + j * 8);
           lm_mma<T>(acc[j], pa[kk], bv[0], bv[1]);
           if (j + 1 < nv) lm_mma<T>(acc[j + 1], pa[kk], bv[2], bv[3]);
+          if constexpr (WIDE) {
+            lm_mma<T>(acc[j], pb[kk], bv[0], bv[1]);
+            if (j + 1 < nv) lm_mma<T>(acc[j + 1], pb[kk], bv[2], bv[3]);
+          }
         }
       }
     }
@@ -371,7 +397,7 @@ attention_latent_mma_kernel(const T* __restrict__ q, int ldq, T* __restrict__ ou
         }
       continue;
     }
-    const float f = (l[j2] > 0.f ? 1.0f / l[j2] : 0.f) * (gate != nullptr ? gate[(size_t)t * H + h] : 1.0f);
+    const float f = softmax_sink_factor(m[j2], l[j2], sink, h) * (gate != nullptr ? gate[(size_t)t * H + h] : 1.0f);
     T* o = out + (size_t)t * ldo + (size_t)h * Dv;
 #pragma unroll
     for (int j = 0; j < NV; ++j)
@@ -397,7 +423,7 @@ FERRUM_API int ferrum_attention_latent_mma(const void* q, int ldq, void* out, in
                                            const int* positions, const int* q_start, int n_reqs, const int* block_table,
                                            int table_width, const void* plane, long long page_stride, int page_size, int H, int Dk,
                                            int Dv, float scale, int window, int single_tokens, float* part, int split_slots,
-                                           int* err_flag, cudaStream_t stream) {
+                                           const float* sink, int* err_flag, int wide, cudaStream_t stream) {
   FERRUM_CHECK_ARG(n_tokens >= 0 && n_reqs > 0 && H > 0, "latent attention: bad sizes T=%d requests=%d H=%d", n_tokens, n_reqs, H);
   FERRUM_CHECK_ARG(ferrum_attention_latent_mma_supported(dtype, Dk, Dv, ldq, ldo, page_stride, q, out, plane),
                    "latent attention (tensor cores): shape Dk=%d Dv=%d or alignment not supported", Dk, Dv);
@@ -411,9 +437,9 @@ FERRUM_API int ferrum_attention_latent_mma(const void* q, int ldq, void* out, in
   const int TT = 16 / HB;
   const int hchunks = (H + HB - 1) / HB;
   const int nvq = Dv / 32;
-#define LM_LAUNCH(NV_, NRT_, TK_)                                                                                              \
+#define LM_LAUNCH_W(NV_, NRT_, TK_, W_)                                                                                        \
   do {                                                                                                                       \
-    const LmSmem s = lm_smem(Dk, NRT_, TK_);                                                                                   \
+    const LmSmem s = lm_smem(Dk, NRT_, TK_, W_);                                                                               \
     const int TQ_ = TT * NRT_;                                                                                               \
     const long long chunks = TQ_ == 1 ? n_tokens : (n_tokens + TQ_ - 1) / TQ_ + n_reqs;                                      \
     const long long ctas = chunks * hchunks;                                                                                 \
@@ -421,17 +447,22 @@ FERRUM_API int ferrum_attention_latent_mma(const void* q, int ldq, void* out, in
     FERRUM_DISPATCH_16BIT(dtype, T, {                                                                                        \
       static int configured = 0;                                                                                             \
       if (configured < s.bytes) {                                                                                            \
-        cudaError_t e = cudaFuncSetAttribute(attention_latent_mma_kernel<T, NV_, NRT_, TK_>,                                      \
+        cudaError_t e = cudaFuncSetAttribute(attention_latent_mma_kernel<T, NV_, NRT_, TK_, W_>,                                  \
                                              cudaFuncAttributeMaxDynamicSharedMemorySize, s.bytes);                          \
         FERRUM_CHECK_ARG(e == cudaSuccess, "latent attention: cannot reserve %d bytes of shared memory: %s", s.bytes,        \
                          cudaGetErrorString(e));                                                                             \
         configured = s.bytes;                                                                                                \
       }                                                                                                                      \
-      launch_kernel(attention_latent_mma_kernel<T, NV_, NRT_, TK_>, dim3((unsigned)ctas, part ? split_slots : 1), dim3(128 * NRT_), \
+      launch_kernel(attention_latent_mma_kernel<T, NV_, NRT_, TK_, W_>, dim3((unsigned)ctas, part ? split_slots : 1), dim3(128 * NRT_), \
                     (size_t)s.bytes, stream, (const T*)q, ldq, (T*)out, ldo, gate, positions, q_start, n_reqs, block_table,    \
                     table_width, (const T*)plane, page_stride, page_size, H, HB, Dk, Dv, scale, window, err_flag, s.DKP,       \
-                    s.off_k, s.off_s, s.off_row, part, split_slots);                                                          \
+                    s.off_k, s.off_s, s.off_row, part, split_slots, sink);                                                          \
     });                                                                                                                      \
+  } while (0)
+#define LM_LAUNCH(NV_, NRT_, TK_)                    \
+  do {                                               \
+    if (wide) LM_LAUNCH_W(NV_, NRT_, TK_, true);     \
+    else LM_LAUNCH_W(NV_, NRT_, TK_, false);         \
   } while (0)
   // Prompt portions: three row tiles (12 warps) on stages of 64 keys where shared memory holds them, else
   // two, else (a very long key row) two on stages of 32 keys.  Single tokens: one row tile; stages of 32
@@ -446,13 +477,13 @@ FERRUM_API int ferrum_attention_latent_mma(const void* q, int ldq, void* out, in
       sms = 148;
   }
   bool big_grid = (long long)n_tokens * hchunks * (part ? split_slots : 1) > 2LL * sms;
-  int fit64 = lm_smem(Dk, 3, 64).bytes <= LM_SMEM_LIMIT ? 3 : (lm_smem(Dk, 2, 64).bytes <= LM_SMEM_LIMIT ? 2 : 0);
+  int fit64 = lm_smem(Dk, 3, 64, wide).bytes <= LM_SMEM_LIMIT ? 3 : (lm_smem(Dk, 2, 64, wide).bytes <= LM_SMEM_LIMIT ? 2 : 0);
   if (g_force_stage == 32) big_grid = true, fit64 = 0;
   if (g_force_stage == 64) big_grid = false;
 #define LM_SHAPES(NV_)                                                          \
   do {                                                                          \
     if (single_tokens) {                                                        \
-      if (big_grid || lm_smem(Dk, 1, 64).bytes > LM_SMEM_LIMIT) LM_LAUNCH(NV_, 1, 32); \
+      if (big_grid || lm_smem(Dk, 1, 64, wide).bytes > LM_SMEM_LIMIT) LM_LAUNCH(NV_, 1, 32); \
       else LM_LAUNCH(NV_, 1, 64);                                               \
     } else if (fit64 == 3) LM_LAUNCH(NV_, 3, 64);                               \
     else if (fit64 == 2) LM_LAUNCH(NV_, 2, 64);                                 \
@@ -463,6 +494,7 @@ FERRUM_API int ferrum_attention_latent_mma(const void* q, int ldq, void* out, in
   else LM_SHAPES(16);
 #undef LM_SHAPES
 #undef LM_LAUNCH
+#undef LM_LAUNCH_W
   FERRUM_CHECK_LAUNCH("attention_latent_mma");
   return 0;
 }

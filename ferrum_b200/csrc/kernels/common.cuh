@@ -159,6 +159,12 @@ __device__ __forceinline__ float glu_swish_clamp(float gate, float up, float lim
   return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
 }
 
+// The activation of an ungated unit: the square of relu.
+__device__ __forceinline__ float relu_squared(float z) {
+  const float r = fmaxf(z, 0.f);
+  return r * r;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -43,6 +43,7 @@ enum TcEpilogue : int {
   TC_SWIGLU = 3,      // out 16-bit [M, ldo] = silu(acc0) * acc1   (DUAL only)
   TC_GEGLU = 4,       // the same with the tanh form of gelu on acc0 (an entry point's argument; the kernels see TC_SWIGLU and glu_act)
   TC_SWISH_CLAMP = 5, // the clamped unit (common.cuh) of acc0 and acc1 with the entry point's glu_limit (likewise)
+  TC_RELU2 = 6,       // out 16-bit [M, ldo] = relu(acc)^2   (the kernels see TC_STORE_BF16 and store_act)
 };
 
 struct TcParams {
@@ -63,7 +64,10 @@ struct TcParams {
   int drop_loads;      // test hook: the producer requests no tile at all, so that the waits for them run out
   int glu_act;         // activation of the gate in the SwiGLU epilogues: 0 silu, 1 gelu (tanh form), 2 the clamped unit
   float glu_limit;     // the clamp of activation 2
+  int store_act;       // what the plain 16-bit store applies: 0 nothing, 1 the square of relu
 };
+
+__device__ __forceinline__ float tc_store_act(float v, const TcParams& p) { return p.store_act ? relu_squared(v) : v; }
 
 // act(gate) of the gated epilogues, float32.
 __device__ __forceinline__ float tc_glu_act(float g, int act) {
@@ -111,7 +115,7 @@ __device__ __forceinline__ void tc_apply16(const TcParams& p, int t_base, int n,
       const bool half = p.half != 0;
 #pragma unroll
       for (int j = 0; j < 16; ++j)
-        if (j < valid) out[j * ld] = bits16(a0[j], half);
+        if (j < valid) out[j * ld] = bits16(tc_store_act(a0[j], p), half);
       break;
     }
     case TC_STORE_F32: {
@@ -716,7 +720,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
           uint16_t* st = (uint16_t*)stage;
           const bool half = p.half != 0;
 #pragma unroll
-          for (int j = 0; j < 32; ++j) st[j * TILE_N + n_local] = bits16(v[j], half);
+          for (int j = 0; j < 32; ++j) st[j * TILE_N + n_local] = bits16(tc_store_act(v[j], p), half);
         }
         stage_send(stage, &tmap_out, p.epilogue == TC_RESIDUAL, n0_cta, t0 + c0);
       } else if (n0_cta + n_local < p.N) {
@@ -966,8 +970,8 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
 #pragma unroll
               for (int k = 0; k < 8; ++k) {
                 uint2 pk;
-                pk.x = pack2_bits(acc[k].x, acc[k].y, p.half != 0);
-                pk.y = pack2_bits(acc[k].z, acc[k].w, p.half != 0);
+                pk.x = pack2_bits(tc_store_act(acc[k].x, p), tc_store_act(acc[k].y, p), p.half != 0);
+                pk.y = pack2_bits(tc_store_act(acc[k].z, p), tc_store_act(acc[k].w, p), p.half != 0);
                 *reinterpret_cast<uint2*>((uint16_t*)stage + (cg + k) * TILE_N + q4) = pk;
               }
             }
@@ -1209,6 +1213,8 @@ FERRUM_API int ferrum_gemm_tc(const void* x, const void* w, void* out, int dtype
   const bool dual = dual_offset > 0;
   const int glu_act = epilogue == TC_GEGLU ? 1 : (epilogue == TC_SWISH_CLAMP ? GLU_SWISH_CLAMP : 0);
   if (epilogue == TC_GEGLU || epilogue == TC_SWISH_CLAMP) epilogue = TC_SWIGLU;
+  const int store_act = epilogue == TC_RELU2;
+  if (epilogue == TC_RELU2) epilogue = TC_STORE_BF16;
   FERRUM_CHECK_ARG(dual == (epilogue == TC_SWIGLU), "gemm_tc: the SwiGLU epilogue needs dual_offset, and only it does");
   FERRUM_CHECK_ARG(epilogue >= 0 && epilogue <= 3, "gemm_tc: unknown epilogue %d", epilogue);
   FERRUM_CHECK_ARG(w_rows >= N + dual_offset, "gemm_tc: w has %d rows, needs %d", w_rows, N + dual_offset);
@@ -1230,6 +1236,7 @@ FERRUM_API int ferrum_gemm_tc(const void* x, const void* w, void* out, int dtype
   p.stream_weights = (M + bt - 1) / bt == 1;  // one token tile: no weight tile is read twice
   p.glu_act = glu_act;
   p.glu_limit = glu_limit;
+  p.store_act = store_act;
   CUtensorMap mw, mx;
   if (dual && M > TILE_N && g_pair_kernel && n_ctas >= 2 && ((uintptr_t)out & 15) == 0 && ldo % 8 == 0) {
     // Two products of many tokens: the pair kernel computes them as one product whose weight
@@ -1700,7 +1707,7 @@ FERRUM_API int ferrum_gemm_tc_grouped_supported(const void* x, const void* w, in
 
 // x [x_rows, ldx] (the first n_rows sorted by expert), w [n_exp, w_rows, K] dense, counts [n_exp] on the device.
 // glu: 0 float32 rows out [n_rows, ldo]; 1 / 2: silu / gelu_tanh of the gate rows times the up rows (rows N + n), 3: the
-// clamped unit of both with glu_limit; out in the operands' type.
+// clamped unit of both with glu_limit; -1: the square of relu, no gate; out in the operands' type.
 FERRUM_API int ferrum_gemm_tc_grouped(const void* x, const void* w, void* out, int dtype, int n_rows, int x_rows, int N, int K,
                                       int ldx, int ldo, int n_exp, int w_rows, const int* counts, int glu, int* err_flag,
                                       float glu_limit, cudaStream_t stream) {
@@ -1710,9 +1717,10 @@ FERRUM_API int ferrum_gemm_tc_grouped(const void* x, const void* w, void* out, i
   if (n_rows == 0) return 0;
   FERRUM_CHECK_ARG(ferrum_gemm_tc_grouped_supported(x, w, n_rows, n_exp, K, ldx), "gemm_tc_grouped: rows must be 16-byte multiples "
                    "on 16-byte boundaries, and at most %d row tiles", GR_MAX_ROW_TILES);
-  FERRUM_CHECK_ARG(ldx >= K && ldo >= N && x_rows >= n_rows && w_rows >= (glu ? 2 * N : N), "gemm_tc_grouped: shapes do not agree");
-  const bool dual = glu != 0;
-  TcParams p{out, nullptr, nullptr, err_flag, n_rows, N, K, ldo, dual ? TC_SWIGLU : TC_STORE_F32, dual ? N : 0, 0};
+  FERRUM_CHECK_ARG(ldx >= K && ldo >= N && x_rows >= n_rows && w_rows >= (glu > 0 ? 2 * N : N), "gemm_tc_grouped: shapes do not agree");
+  const bool dual = glu > 0;
+  TcParams p{out, nullptr, nullptr, err_flag, n_rows, N, K, ldo, dual ? TC_SWIGLU : (glu < 0 ? TC_STORE_BF16 : TC_STORE_F32), dual ? N : 0, 0};
+  p.store_act = glu < 0;
   p.half = dtype == FERRUM_F16;
   p.wait_cycles = g_wait_cycles;
   p.drop_loads = g_drop_loads;

@@ -10,16 +10,24 @@
 //   cache row (normalised latent, rotated key part) written to the token's page, and the sigmoid
 //   of the output-gate logits.
 // latent_q_rope: the rotated part of every query head, moved behind the folded part.
-// attention_latent: the attention itself, float32 arithmetic, for float32 and 16-bit storage.
+// attention_latent: the attention itself, float32 arithmetic, for float32 and 16-bit storage.  With `sink`
+//   (one float per head) exp(sink_h) joins the denominator of head h's softmax: a key without a value, seen by
+//   every query.  It enters once, where a row's maximum and sum are final (in the fold when key ranges are split).
+// pairing: 1 pairs elements (i, i + dims/2) of the rotated part, 0 neighbours (2i, 2i + 1).
 #include "common.cuh"
 #include "partials.cuh"
+#include "softmax_sink.cuh"
 
 constexpr int LAT_THREADS = 256;
 
-// pairing (i, i + dims/2) of the first `dims` elements; the others pass unchanged
-__device__ __forceinline__ float latent_rotated(const float* v, int i, int dims, const float* cs) {
+// element i of v with its first `dims` elements turned; the others pass unchanged
+__device__ __forceinline__ float latent_rotated(const float* v, int i, int dims, const float* cs, int pairing) {
   const int half = dims >> 1;
   if (i >= dims) return v[i];
+  if (pairing == 0) {
+    const float c = cs[i & ~1], s = cs[i | 1];
+    return (i & 1) ? v[i] * c + v[i - 1] * s : v[i] * c - v[i + 1] * s;
+  }
   if (i < half) return v[i] * cs[2 * i] - v[i + half] * cs[2 * i + 1];
   const int k = i - half;
   return v[i] * cs[2 * k] + v[k] * cs[2 * k + 1];
@@ -30,7 +38,7 @@ __global__ void __launch_bounds__(LAT_THREADS)
 latent_prep_kernel(const float* __restrict__ proj, int ld, int off_q, int q_rank, const float* __restrict__ wq, int off_kv, int kv_rank,
                    int rot_dim, const float* __restrict__ wkv, int off_gate, int n_gate, const int* __restrict__ positions,
                    const int* __restrict__ req_of_token, const int* __restrict__ block_table, int table_width,
-                   const float* __restrict__ cos_sin, int n_pos, int rope_dims, T* __restrict__ plane, long long page_stride,
+                   const float* __restrict__ cos_sin, int n_pos, int rope_dims, int pairing, T* __restrict__ plane, long long page_stride,
                    int page_size, T* __restrict__ cq, int ld_cq, float* __restrict__ gate, float eps, int* __restrict__ err,
                    int n_in, const PartialLayout L) {
   __shared__ float red[32];
@@ -75,7 +83,7 @@ latent_prep_kernel(const float* __restrict__ proj, int ld, int off_q, int q_rank
   for (int i = threadIdx.x; i < kv_rank; i += blockDim.x) dst[i] = from_f32<T>(p[i] * inv * wkv[i]);
   const float* cs = rope_dims > 0 ? cos_sin + (size_t)pos * rope_dims : nullptr;      // [dims/2][2]
   for (int i = threadIdx.x; i < rot_dim; i += blockDim.x)
-    dst[kv_rank + i] = from_f32<T>(rope_dims > 0 ? latent_rotated(p + kv_rank, i, rope_dims, cs) : p[kv_rank + i]);
+    dst[kv_rank + i] = from_f32<T>(rope_dims > 0 ? latent_rotated(p + kv_rank, i, rope_dims, cs, pairing) : p[kv_rank + i]);
 }
 
 // With `partials` (a product left in deferred mode, see partials.cuh) the projections are summed from
@@ -87,7 +95,7 @@ latent_prep_kernel(const float* __restrict__ proj, int ld, int off_q, int q_rank
 FERRUM_API int ferrum_latent_prep(const float* proj, int ld, int n_tokens, int off_q, int q_rank, const float* wq, int off_kv,
                                   int kv_rank, int rot_dim, const float* wkv, int off_gate, int n_gate, const int* positions,
                                   const int* req_of_token, const int* block_table, int table_width, const float* cos_sin,
-                                  int n_pos, int rope_dims, void* plane, long long page_stride, int page_size, void* cq,
+                                  int n_pos, int rope_dims, int pairing, void* plane, long long page_stride, int page_size, void* cq,
                                   int ld_cq, int dtype, float* gate, float eps, int* err_flag, const float* partials,
                                   const int* layout, cudaStream_t stream) {
   FERRUM_CHECK_ARG(n_tokens >= 0 && q_rank >= 0 && kv_rank > 0 && rot_dim >= 0 && n_gate >= 0, "latent prep: bad sizes");
@@ -110,7 +118,7 @@ FERRUM_API int ferrum_latent_prep(const float* proj, int ld, int n_tokens, int o
       FERRUM_CHECK_ARG(e == cudaSuccess, "latent prep: cannot reserve %d bytes of shared memory: %s", n_in * 4, cudaGetErrorString(e));
     }
     launch_kernel(latent_prep_kernel<T>, n_tokens, LAT_THREADS, (size_t)n_in * 4, stream, proj, ld, off_q, q_rank, wq, off_kv, kv_rank,
-                  rot_dim, wkv, off_gate, n_gate, positions, req_of_token, block_table, table_width, cos_sin, n_pos, rope_dims,
+                  rot_dim, wkv, off_gate, n_gate, positions, req_of_token, block_table, table_width, cos_sin, n_pos, rope_dims, pairing,
                   (T*)plane, page_stride, page_size, (T*)cq, ld_cq, gate, eps, err_flag, n_in, L);
   });
   FERRUM_CHECK_LAUNCH("latent_prep");
@@ -123,7 +131,7 @@ FERRUM_API int ferrum_latent_prep(const float* proj, int ld, int n_tokens, int o
 template <typename T>
 __global__ void __launch_bounds__(LAT_THREADS)
 latent_q_rope_kernel(const T* __restrict__ q, int ldq, T* __restrict__ qf, int ldf, const int* __restrict__ positions,
-                     const float* __restrict__ cos_sin, int n_pos, int rope_dims, int H, int Dn, int Rr, int R, int* __restrict__ err) {
+                     const float* __restrict__ cos_sin, int n_pos, int rope_dims, int pairing, int H, int Dn, int Rr, int R, int* __restrict__ err) {
   pdl_launch();
   pdl_wait();
   const int t = blockIdx.x;
@@ -139,7 +147,8 @@ latent_q_rope_kernel(const T* __restrict__ q, int ldq, T* __restrict__ qf, int l
     const T* src = q + (size_t)t * ldq + (size_t)h * (Dn + Rr) + Dn;
     float v = to_f32<T>(src[i]);
     if (i < rope_dims) {
-      if (i < half) v = v * cs[2 * i] - to_f32<T>(src[i + half]) * cs[2 * i + 1];
+      if (pairing == 0) v = (i & 1) ? v * cs[i - 1] + to_f32<T>(src[i - 1]) * cs[i] : v * cs[i] - to_f32<T>(src[i + 1]) * cs[i + 1];
+      else if (i < half) v = v * cs[2 * i] - to_f32<T>(src[i + half]) * cs[2 * i + 1];
       else v = v * cs[2 * (i - half)] + to_f32<T>(src[i - half]) * cs[2 * (i - half) + 1];
     }
     qf[(size_t)t * ldf + (size_t)h * (R + Rr) + R + i] = from_f32<T>(v);
@@ -147,14 +156,14 @@ latent_q_rope_kernel(const T* __restrict__ q, int ldq, T* __restrict__ qf, int l
 }
 
 FERRUM_API int ferrum_latent_q_rope(const void* q, int ldq, void* qf, int ldf, int dtype, int n_tokens, const int* positions,
-                                    const float* cos_sin, int n_pos, int rope_dims, int H, int Dn, int Rr, int R, int* err_flag,
+                                    const float* cos_sin, int n_pos, int rope_dims, int pairing, int H, int Dn, int Rr, int R, int* err_flag,
                                     cudaStream_t stream) {
   FERRUM_CHECK_ARG(n_tokens >= 0 && H > 0 && Dn >= 0 && Rr >= 0 && R > 0, "latent q rope: bad sizes");
   FERRUM_CHECK_ARG(rope_dims >= 0 && rope_dims % 2 == 0 && rope_dims <= Rr, "latent q rope: %d rotated dimensions of %d", rope_dims, Rr);
   FERRUM_CHECK_ARG(ldq >= H * (Dn + Rr) && ldf >= H * (R + Rr), "latent q rope: a row stride is too short");
   if (n_tokens == 0 || Rr == 0) return 0;
   FERRUM_DISPATCH_DTYPE(dtype, T, launch_kernel(latent_q_rope_kernel<T>, n_tokens, LAT_THREADS, 0, stream, (const T*)q, ldq, (T*)qf, ldf,
-                                                positions, cos_sin, n_pos, rope_dims, H, Dn, Rr, R, err_flag));
+                                                positions, cos_sin, n_pos, rope_dims, pairing, H, Dn, Rr, R, err_flag));
   FERRUM_CHECK_LAUNCH("latent_q_rope");
   return 0;
 }
@@ -222,7 +231,7 @@ attention_latent_kernel(const T* __restrict__ q, int ldq, T* __restrict__ out, i
                         const int* __restrict__ positions, const int* __restrict__ q_start, int n_reqs,
                         const int* __restrict__ block_table, int table_width, const T* __restrict__ plane, long long page_stride,
                         int page_size, int H, int Dk, int Dv, float scale, int window, int* __restrict__ err, int vec, int TK,
-                        int DK8, int off_q, int off_p, int off_row, float* __restrict__ part, int split_slots) {
+                        int DK8, int off_q, int off_p, int off_row, float* __restrict__ part, int split_slots, const float* __restrict__ sink) {
   constexpr int TW = LAT_WARPS / HW, TQ = TH * TW;
   extern __shared__ __align__(16) float lat_sm[];
   const int KS = DK8 + 4;
@@ -435,7 +444,7 @@ attention_latent_kernel(const T* __restrict__ q, int ldq, T* __restrict__ out, i
       }
       continue;
     }
-    const float f = (l[i] > 0.f ? 1.0f / l[i] : 0.f) * (gate != nullptr ? gate[(size_t)t * H + h] : 1.0f);
+    const float f = softmax_sink_factor(m[i], l[i], sink, h) * (gate != nullptr ? gate[(size_t)t * H + h] : 1.0f);
 #pragma unroll
     for (int e = 0; e < DVI; ++e) {
       const int d = lane + 32 * e;
@@ -452,9 +461,10 @@ constexpr int LAT_COMB_THREADS = 128, LAT_COMB_MAX = 1024;
 template <typename T>
 __global__ void __launch_bounds__(LAT_COMB_THREADS)
 attention_latent_combine_kernel(T* __restrict__ out, int ldo, const float* __restrict__ part, const float* __restrict__ gate,
-                                const int* __restrict__ positions, int H, int Dv, int window, int split_slots) {
+                                const int* __restrict__ positions, int H, int Dv, int window, int split_slots,
+                                const float* __restrict__ sink) {
   __shared__ float factor[LAT_COMB_MAX];
-  __shared__ float total;
+  __shared__ float total, top;
   pdl_launch();
   pdl_wait();
   const int t = blockIdx.x, h = blockIdx.y;
@@ -474,11 +484,13 @@ attention_latent_combine_kernel(T* __restrict__ out, int ldo, const float* __res
       sum += base[(size_t)s * (Dv + 2) + 1] * f;
     }
     sum = warp_sum(sum);
-    if (threadIdx.x == 0) total = sum;
+    if (threadIdx.x == 0) {
+      total = sum;
+      top = mx;
+    }
   }
   __syncthreads();
-  const float L = total;
-  const float f = (L > 0.f ? 1.0f / L : 0.f) * (gate != nullptr ? gate[(size_t)t * H + h] : 1.0f);
+  const float f = softmax_sink_factor(top, total, sink, h) * (gate != nullptr ? gate[(size_t)t * H + h] : 1.0f);
   for (int d = threadIdx.x; d < Dv; d += LAT_COMB_THREADS) {
     float o = 0.f;
     for (int s = 0; s < n; ++s) o = fmaf(base[(size_t)s * (Dv + 2) + 2 + d], factor[s], o);
@@ -490,12 +502,13 @@ FERRUM_API int ferrum_attention_latent_split() { return LAT_SPLIT; }
 
 // out[t, h] = gate[t, h] * (the fold of the splits' partials [t][h][slot][Dv + 2] in ascending key order).
 FERRUM_API int ferrum_attention_latent_combine(void* out, int ldo, int dtype, const float* part, const float* gate, int n_tokens,
-                                               const int* positions, int H, int Dv, int window, int split_slots, cudaStream_t stream) {
+                                               const int* positions, int H, int Dv, int window, int split_slots, const float* sink,
+                                               cudaStream_t stream) {
   FERRUM_CHECK_ARG(n_tokens >= 0 && H > 0 && H <= 65535 && Dv > 0 && split_slots > 0 && split_slots <= LAT_COMB_MAX && part != nullptr,
                    "latent attention merge: bad arguments (at most %d splits)", LAT_COMB_MAX);
   if (n_tokens == 0) return 0;
   FERRUM_DISPATCH_DTYPE(dtype, T, launch_kernel(attention_latent_combine_kernel<T>, dim3(n_tokens, H), dim3(LAT_COMB_THREADS), 0, stream, (T*)out, ldo,
-                                                part, gate, positions, H, Dv, window, split_slots));
+                                                part, gate, positions, H, Dv, window, split_slots, sink));
   FERRUM_CHECK_LAUNCH("attention_latent_combine");
   return 0;
 }
@@ -510,7 +523,7 @@ FERRUM_API int ferrum_attention_latent(const void* q, int ldq, void* out, int ld
                                        const int* positions, const int* q_start, int n_reqs, const int* block_table,
                                        int table_width, const void* plane, long long page_stride, int page_size, int H, int Dk,
                                        int Dv, float scale, int window, int single_tokens, float* part, int split_slots,
-                                       int* err_flag, cudaStream_t stream) {
+                                       const float* sink, int* err_flag, cudaStream_t stream) {
   FERRUM_CHECK_ARG(part == nullptr || (single_tokens && split_slots > 0 && split_slots <= 65535),
                    "latent attention: key splits are for steps of single tokens (slots %d)", split_slots);
   FERRUM_CHECK_ARG(n_tokens >= 0 && n_reqs > 0 && H > 0, "latent attention: bad sizes T=%d requests=%d H=%d", n_tokens, n_reqs, H);
@@ -549,7 +562,7 @@ FERRUM_API int ferrum_attention_latent(const void* q, int ldq, void* out, int ld
                     dim3(LAT_WARPS * 32), (size_t)s.bytes,                                                                  \
                     stream, (const T*)q, ldq, (T*)out, ldo, gate, positions, q_start, n_reqs, block_table, table_width,     \
                     (const T*)plane, page_stride, page_size, H, Dk, Dv, scale, window, err_flag, vec, TK, s.DK8, s.off_q,    \
-                    s.off_p, s.off_row, part, split_slots);                                                                 \
+                    s.off_p, s.off_row, part, split_slots, sink);                                                                 \
     });                                                                                                                     \
   } while (0)
 #define LAT_SHAPES(DVI_)                               \
@@ -568,7 +581,7 @@ FERRUM_API int ferrum_attention_latent(const void* q, int ldq, void* out, int ld
 #undef LAT_SHAPES
 #undef LAT_LAUNCH
   FERRUM_CHECK_LAUNCH("attention_latent");
-  if (part != nullptr) return ferrum_attention_latent_combine(out, ldo, dtype, part, gate, n_tokens, positions, H, Dv, window, split_slots, stream);
+  if (part != nullptr) return ferrum_attention_latent_combine(out, ldo, dtype, part, gate, n_tokens, positions, H, Dv, window, split_slots, sink, stream);
   return 0;
 }
 

@@ -6,7 +6,9 @@
 //             A correction vector may be added to the scores for the choice alone (the weights stay the
 //             plain scores), the weights may be multiplied by a constant, and the last router outputs may
 //             be identity experts (numbers n_real .. n_exp - 1: no matrices, no rows in the sorted buffer;
-//             the consumer adds weight * the token's own input for them).
+//             the consumer adds weight * the token's own input for them).  With groups (experts in equal
+//             groups of neighbours) only the experts of the best groups can be chosen, a group being worth the
+//             sum of its two largest choice scores.
 // moe_gather  one block per (token, choice): the token's input row, multiplied by the choice's weight
 //             where the design scales the expert's INPUT, goes to its place in a buffer sorted by
 //             expert (row = first row of the expert's group + the place taken above).
@@ -14,7 +16,8 @@
 //             of rows of ONE expert (it finds expert and rows from the counters, so nothing about the
 //             routing passes through the host) and a tile of output features.  Two epilogues: the
 //             gated activation act(gate) * up from weight rows n and F + n, stored in the compute type;
-//             or float32 rows.  float32 accumulation in an order that depends on K and on the kernel
+//             or float32 rows; or, for units without a gate, the activation of C itself in the compute type.
+//             float32 accumulation in an order that depends on K and on the kernel
 //             only: a row's result does not depend on the rows it shares a tile with.  Three kernels:
 //             tiles on the CUDA cores (float32, and 16-bit rows that are no 16-byte multiples), a
 //             warp per feature when an expert has a few rows (the same types, decoding), and tiles on
@@ -36,7 +39,82 @@ struct MoeRouter {
   const float* correction;   // [n_exp] or null
   float weight_scale;
   const float* bias;         // [n_exp] or null
+  int groups, keep;          // groups > keep > 0: only experts of the `keep` best of `groups` equal groups can be chosen
+  float renorm_eps;          // added to the sum of the chosen scores before the division
 };
+
+// The picks of experts outside the best groups become minus infinity (a tie between groups goes to the lower one).
+__device__ __forceinline__ void moe_keep_groups(const MoeRouter& R, int lane, float (&pick)[MOE_MAX_EXPERTS / 32]) {
+  constexpr int PER = MOE_MAX_EXPERTS / 32;
+  const int size = R.n_exp / R.groups;
+  float worth[PER];                         // lane l holds what groups l, l + 32, ... are worth
+#pragma unroll
+  for (int i = 0; i < PER; ++i) worth[i] = -INFINITY;
+  for (int g = 0; g < R.groups; ++g) {
+    float a = -INFINITY, b = -INFINITY;     // the two largest picks of the group
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const int e = lane + 32 * i;
+      if (e >= g * size && e < (g + 1) * size) {
+        const float v = pick[i];
+        if (v > a) b = a, a = v;
+        else if (v > b) b = v;
+      }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float oa = __shfl_xor_sync(0xffffffffu, a, o), ob = __shfl_xor_sync(0xffffffffu, b, o);
+      b = fmaxf(fminf(a, oa), fmaxf(b, ob));
+      a = fmaxf(a, oa);
+    }
+    const float sum = size > 1 ? a + b : a;
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (lane + 32 * i == g) worth[i] = sum;
+  }
+  unsigned kept[PER];                       // bit g % 32 of word g / 32, the same in every lane
+#pragma unroll
+  for (int i = 0; i < PER; ++i) kept[i] = 0u;
+  for (int k = 0; k < R.keep; ++k) {
+    float best = -INFINITY;
+    int best_g = 0x7fffffff;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const int g = lane + 32 * i;
+      const bool taken = (kept[i] >> lane) & 1u;
+      if (g < R.groups && !taken && (worth[i] > best || best_g == 0x7fffffff)) {
+        best = worth[i];
+        best_g = g;
+      }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int og = __shfl_xor_sync(0xffffffffu, best_g, o);
+      if (og != 0x7fffffff && (best_g == 0x7fffffff || ob > best || (ob == best && og < best_g))) {
+        best = ob;
+        best_g = og;
+      }
+    }
+    // (a NaN compares false both ways: lanes could disagree, so every lane takes lane 0's answer)
+    best_g = __shfl_sync(0xffffffffu, best_g, 0);
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (best_g >> 5 == i) kept[i] |= 1u << (best_g & 31);
+  }
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int e = lane + 32 * i;
+    if (e < R.n_exp) {
+      const int g = e / size;
+      unsigned word = 0u;
+#pragma unroll
+      for (int j = 0; j < PER; ++j)
+        if (g >> 5 == j) word = kept[j];
+      if (!((word >> (g & 31)) & 1u)) pick[i] = -INFINITY;
+    }
+  }
+}
 __device__ __forceinline__ void moe_choose(const MoeRouter& R, int t, int lane, int (&chosen_e)[MOE_MAX_TOP], float (&chosen_w)[MOE_MAX_TOP]) {
   const float* const logits = R.logits;
   const float* const bias = R.bias;
@@ -74,6 +152,7 @@ __device__ __forceinline__ void moe_choose(const MoeRouter& R, int t, int lane, 
     const int e = lane + 32 * i;
     pick[i] = (correction != nullptr && e < n_exp) ? s[i] + correction[e] : s[i];
   }
+  if (R.groups > R.keep && R.keep > 0) moe_keep_groups(R, lane, pick);
   float total = 0.f;
   for (int j = 0; j < top; ++j) {
     float best = -INFINITY, best_s = 0.f;
@@ -116,7 +195,7 @@ __device__ __forceinline__ void moe_choose(const MoeRouter& R, int t, int lane, 
   }
   for (int j = 0; j < top; ++j) {
     if (chosen_e[j] >= n_exp) chosen_e[j] = 0;      // (all scores NaN: expert 0 with a NaN weight)
-    chosen_w[j] = (R.renormalize ? chosen_w[j] / total : chosen_w[j]) * R.weight_scale;
+    chosen_w[j] = (R.renormalize ? chosen_w[j] / (total + R.renorm_eps) : chosen_w[j]) * R.weight_scale;
   }
 }
 
@@ -217,6 +296,8 @@ __device__ __forceinline__ float moe_act(float z, int act) {
   if (act == 1) return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
   return z / (1.f + expf(-z));
 }
+// Activation code of units without a gate (the product's `act` in the form that is not gated): the square of relu.
+constexpr int UNIT_RELU2 = 16;
 // What the gated epilogue stores for a gate value and an up value (act 2: the clamped unit of common.cuh).
 __device__ __forceinline__ float moe_glu(float g, float u, int act, float limit) {
   if (act == GLU_SWISH_CLAMP) return glu_swish_clamp(g, u, limit);
@@ -308,6 +389,7 @@ moe_gemm_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, int w
       const int n = n0 + tx * TN + j;
       if (n >= N) continue;
       if (GLU) reinterpret_cast<T*>(out)[row * ldo + n] = from_f32<T>(moe_glu(acc[0][i][j], acc[1][i][j], act, limit));
+      else if (act == UNIT_RELU2) reinterpret_cast<T*>(out)[row * ldo + n] = from_f32<T>(relu_squared(acc[0][i][j]));
       else reinterpret_cast<float*>(out)[row * ldo + n] = acc[0][i][j];
     }
   }
@@ -399,6 +481,7 @@ moe_gemm_skinny_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W
   if (lane < rows) {
     const size_t o = (size_t)(row0 + lane) * ldo + n;
     if (GLU) reinterpret_cast<T*>(out)[o] = from_f32<T>(moe_glu(r0, r1, act, limit));
+    else if (act == UNIT_RELU2) reinterpret_cast<T*>(out)[o] = from_f32<T>(relu_squared(r0));
     else reinterpret_cast<float*>(out)[o] = r0;
   }
 }
@@ -598,6 +681,7 @@ moe_gemm_mma_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, i
           const int n = n0 + wn * (NI * 8) + j * 8 + (lane & 3) * 2 + c;
           if (n >= N) continue;
           if (GLU) reinterpret_cast<T*>(out)[o + n] = from_f32<T>(moe_glu(acc[0][i][j][h * 2 + c], acc[NB - 1][i][j][h * 2 + c], act, limit));
+          else if (act == UNIT_RELU2) reinterpret_cast<T*>(out)[o + n] = from_f32<T>(relu_squared(acc[0][i][j][h * 2 + c]));
           else reinterpret_cast<float*>(out)[o + n] = acc[0][i][j][h * 2 + c];
         }
     }
@@ -742,17 +826,20 @@ FERRUM_API int ferrum_moe_max_top() { return MOE_MAX_TOP; }
 FERRUM_API int ferrum_moe_route(const float* logits, int ldz, int n_tokens, int n_exp, int top, int score_kind,
                                 int renormalize, const void* x, int ldx, int E, int dtype, int scale_input, int* expert_of,
                                 int* rank_of, float* weight_of, int* counts, void* xg, int* row_of, const float* correction,
-                                float weight_scale, int n_identity, const float* bias, cudaStream_t stream) {
+                                float weight_scale, int n_identity, const float* bias, int groups, int keep, float renorm_eps,
+                                cudaStream_t stream) {
   FERRUM_CHECK_ARG(score_kind >= MOE_SIGMOID && score_kind <= MOE_CHOSEN_SOFTMAX && (score_kind != MOE_CHOSEN_SOFTMAX || correction == nullptr),
                    "moe_route: a softmax over the chosen logits takes no correction");
   FERRUM_CHECK_ARG(n_exp > 0 && n_exp <= MOE_MAX_EXPERTS && top > 0 && top <= MOE_MAX_TOP && top <= n_exp,
                    "moe_route: %d experts, %d per token are outside the kernel's limits (%d, %d)", n_exp, top, MOE_MAX_EXPERTS, MOE_MAX_TOP);
   FERRUM_CHECK_ARG(n_identity >= 0 && n_identity < n_exp, "moe_route: %d identity experts among %d router outputs", n_identity, n_exp);
   FERRUM_CHECK_ARG(n_identity == 0 || !scale_input, "moe_route: identity experts go with weights on the experts' results");
+  FERRUM_CHECK_ARG(groups == 0 || (groups > 0 && keep > 0 && keep <= groups && n_exp % groups == 0 && top <= n_exp / groups * keep),
+                   "moe_route: %d of %d experts in %d groups of which %d are kept", top, n_exp, groups, keep);
   const int n_real = n_exp - n_identity;
   FERRUM_CHECK_ARG(ldz >= n_exp && ldx >= E && E > 0, "moe_route: rows are shorter than their contents");
   if (n_tokens == 0) return 0;
-  const MoeRouter R{logits, ldz, n_exp, top, score_kind, renormalize, correction, weight_scale, bias};
+  const MoeRouter R{logits, ldz, n_exp, top, score_kind, renormalize, correction, weight_scale, bias, groups, keep, renorm_eps};
   if (n_tokens <= MOE_FEW_TOKENS && n_tokens * top <= MOE_FEW_PAIRS) {
     FERRUM_DISPATCH_DTYPE(dtype, T, (moe_route_few_kernel<T><<<n_tokens * top, MOE_FEW_PAIRS, 0, stream>>>(
         R, n_tokens, expert_of, rank_of, weight_of, counts, n_real, (const T*)x, ldx, E, scale_input, (T*)xg, row_of)));
@@ -770,7 +857,8 @@ FERRUM_API int ferrum_moe_route(const float* logits, int ldz, int n_tokens, int 
 }
 
 // n_rows: the sorted rows (tokens x top).  glu != 0: W holds gate rows 0..N-1 and up rows N..2N-1 per expert
-// (w_rows = 2N), out is [n_rows][ldo] in the compute type; else out is float32.
+// (w_rows = 2N), out is [n_rows][ldo] in the compute type; else out is float32, or with act UNIT_RELU2 (16) the activation
+// of the product in the compute type.
 FERRUM_API int ferrum_moe_gemm(const void* A, int lda, const void* W, int w_rows, int K, int N, int n_exp, const int* counts,
                                int n_rows, int dtype, int glu, int act, float limit, void* out, int ldo, cudaStream_t stream) {
   FERRUM_CHECK_ARG(K > 0 && N > 0 && lda >= K && ldo >= N && w_rows >= (glu ? 2 * N : N), "moe_gemm: shapes do not agree");

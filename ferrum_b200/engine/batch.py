@@ -163,6 +163,8 @@ class StepContext:
         # A branch whose normed result joins the residual rows leaves that sum to the norm that reads them next:
         # (residual tensor, ops.PendingAdd) or None.
         self.pending_add = None
+        # A routed feed-forward's expert rows whose weighted sum the next norm adds: (residual tensor, ops.ExpertSum) or None.
+        self.pending_experts = None
         self.defer_residuals = True
         self.defer_swiglu = True
         self.h2d_bytes = 0            # bytes copied to the device by the last fill
@@ -253,6 +255,7 @@ class StepContext:
         self.pending_residual = None
         self.pending_streams = None
         self.pending_add = None
+        self.pending_experts = None
 
     def buffers_generation(self):
         """Changes whenever a buffer that kernels read may have moved (a captured graph is stale then)."""
@@ -290,6 +293,22 @@ class StepContext:
             from ..ops import lib as ops
             self.pending_add = None
             ops.norm_scaled_add(p[0], p[1].y, p[1].w, p[1].mult, p[1].eps, self.n_tokens, partials=p[1].partials)
+        p = self.pending_experts
+        if p is not None:
+            from ..ops import lib as ops
+            self.pending_experts = None
+            ops.moe_combine(p[1].rows, p[1].row_of, p[1].top, self.n_tokens, p[0], weight_of=p[1].weight_of, accumulate=True)
+
+    def take_pending_experts(self, h):
+        """For a norm about to read `h`: the expert rows whose sum it must add first, or None."""
+        p = self.pending_experts
+        if p is None:
+            return None
+        if p[0].data_ptr() == h.data_ptr():
+            self.pending_experts = None
+            return p[1]
+        self.flush_residual()
+        return None
 
     def take_pending_add(self, h):
         """For a norm about to read all rows of `h`: the branch it must add first, or None."""
@@ -318,6 +337,7 @@ class StepContext:
         self.pending_residual = None
         self.pending_streams = None
         self.pending_add = None
+        self.pending_experts = None
 
     # ------------------------------------------------------------------ scratch
     def buf(self, name, shape, dtype):

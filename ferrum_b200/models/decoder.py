@@ -16,7 +16,7 @@ import os
 
 import torch
 
-from ..parts.base import Part
+from ..parts.base import CacheNeed, Part
 
 # FERRUM_NVTX=1: every step and every run of a block is an NVTX range (for a system profiler's timeline)
 NVTX = os.environ.get("FERRUM_NVTX", "0") == "1"
@@ -75,6 +75,10 @@ class DecoderModel(Part):
             out.append(b.cache_need() if hasattr(b, "cache_need") else b.mixer.cache_need())
         return out
 
+    def embedding_need(self):
+        """What the embedding keeps per request beside the runs of the schedule (a `CacheNeed`)."""
+        return self.embedding.cache_need() if hasattr(self.embedding, "cache_need") else CacheNeed()
+
     @property
     def n_vocab(self):
         return self.head.n_vocab
@@ -88,7 +92,8 @@ class DecoderModel(Part):
     def forward(self, ctx, cache):
         """Run the batch described by ctx; returns float32 logits [want_capacity, V] whose
         first ctx.n_want rows are valid, or None when nothing is wanted."""
-        h = self.embedding.forward(ctx)
+        state = cache.embedding_state
+        h = self.embedding.forward(ctx) if state is None else self.embedding.forward(ctx, state)
         if self.position is not None:
             self.position.on_embedding(h, ctx)
         for k, run in enumerate(self.schedule):

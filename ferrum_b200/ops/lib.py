@@ -22,11 +22,11 @@ _DT = {torch.float32: F32, torch.bfloat16: BF16, torch.float16: F16}
 SIXTEEN_BIT = (torch.bfloat16, torch.float16)       # the tensor-core kernels take either
 
 EPI_STORE, EPI_STORE_F32, EPI_RESIDUAL = 0, 1, 2                       # generic product
-TC_STORE_BF16, TC_STORE_F32, TC_RESIDUAL, TC_SWIGLU, TC_GEGLU, TC_SWISH_CLAMP = 0, 1, 2, 3, 4, 5   # tcgen05 product (GEGLU: SWIGLU with gelu_tanh on the gate; SWISH_CLAMP: the clamped unit)
+TC_STORE_BF16, TC_STORE_F32, TC_RESIDUAL, TC_SWIGLU, TC_GEGLU, TC_SWISH_CLAMP, TC_RELU2 = 0, 1, 2, 3, 4, 5, 6   # tcgen05 product (GEGLU: SWIGLU with gelu_tanh on the gate; SWISH_CLAMP: the clamped unit; RELU2: the square of relu, no gate)
 
 _lib = None
 _lock = threading.Lock()
-ABI = 18
+ABI = 19
 
 
 def lib():
@@ -247,6 +247,21 @@ def embedding_norm(table, ids, w, eps, out, err, copy=None):
                                        _stream()), "embedding_norm")
 
 
+def embedding_bigram(table, pairs, ctx, mul_prev, mul_cur, last_id, out, scale=1.0):
+    """out[t] = scale * table[id] + pairs[row], float32, with row = (id before * mul_prev + id * mul_cur) mod (rows of
+    pairs - 1) and the last row of pairs for a sequence's first token.  last_id (int32 [slots]): the id before a
+    portion's first token; receives the portion's last id."""
+    _need(table, None, "table", 2); _need(pairs, table.dtype, "pairs", 2); _need(out, torch.float32, "out", 2); _need(last_id, torch.int32, "last_id")
+    V, E = table.shape
+    T = ctx.n_tokens
+    if out.shape[0] < T or out.shape[1] != E or pairs.shape[1] != E or pairs.shape[0] < 2 or not all(t.is_contiguous() for t in (table, pairs, out, last_id)):
+        raise KernelError("embedding_bigram: shapes do not agree")
+    _check(lib().ferrum_embedding_bigram(_ptr(table), c_int(V), c_float(scale), _ptr(pairs), c_int(pairs.shape[0] - 1), c_longlong(mul_prev),
+                                         c_longlong(mul_cur), dtype_code(table.dtype), _ptr(ctx.token_ids), _ptr(ctx.positions),
+                                         _ptr(ctx.req_of_token), _ptr(ctx.q_start), _ptr(ctx.slots), _ptr(last_id), _ptr(out), c_int(T),
+                                         c_int(E), _ptr(ctx.err), _stream()), "embedding_bigram")
+
+
 class Partials:
     """A product that the tensor-core kernel left as float32 partials (see gemm_tc_deferred):
     the workspace that holds them and the four numbers a consumer needs to sum them."""
@@ -262,6 +277,55 @@ class PendingAdd:
 
     def __init__(self, y, w, mult, eps, partials=None):
         self.y, self.w, self.mult, self.eps, self.partials = y, w, mult, eps, partials
+
+
+class ExpertSum:
+    """A routed feed-forward's result before the sum: row_of[t * top + j] names the row of `rows` that holds token t's j-th
+    choice (-1: none), weight_of its weight (None: the rows are weighted already)."""
+
+    def __init__(self, rows, row_of, top, weight_of):
+        self.rows, self.row_of, self.top, self.weight_of = rows, row_of, top, weight_of
+
+
+def dyn_tanh(x, alpha, w, b, out, rows=None, n_rows=None, partials=None, experts=None):
+    """out[r] = tanh(alpha * x[rows[r] if rows else r]) * w + b; x float32, alpha one float on the device.  With `partials` (a
+    deferred residual product) or `experts` (an `ExpertSum`) the rows of x first get that sum added, in place."""
+    _need(x, torch.float32, "x", 2); _need(out, None, "out", 2); _need(alpha, torch.float32, "alpha")
+    E = x.shape[1]
+    if n_rows is None:
+        n_rows = rows.shape[0] if rows is not None else x.shape[0]
+    for t in (w, b):
+        _need(t, torch.float32, "dyn_tanh vector", 1)
+    if w.shape[0] != E or b.shape[0] != E or alpha.numel() != 1 or out.shape[1] != E or out.shape[0] < n_rows or not x.is_contiguous() or not out.is_contiguous():
+        raise KernelError("dyn_tanh: shapes do not agree")
+    if rows is not None:
+        _need(rows, torch.int32, "rows", 1)
+    if partials is None:
+        global _work
+        if _profile is not None:
+            _work = (n_rows * E * (4 + out.element_size() + (4 * experts.top + 4 if experts is not None else 0)), 0.0)
+    ex = experts if experts is not None else ExpertSum(None, None, 0, None)
+    _check(lib().ferrum_dyn_tanh(_ptr(x), _ptr(alpha), _ptr(w), _ptr(b), _ptr(out), dtype_code(out.dtype), _ptr(rows), c_int(n_rows), c_int(E),
+                                 _ptr(partials.workspace if partials is not None else None), partials._c if partials is not None else None,
+                                 _ptr(ex.rows), c_int(ex.rows.stride(0) if ex.rows is not None else 0), _ptr(ex.row_of), _ptr(ex.weight_of),
+                                 c_int(ex.top), _stream()), "dyn_tanh")
+
+
+UNIT_ACTS = {"relu2": 16}        # activations of units without a gate: the square of relu
+
+
+def unit_act(x, out, n_tokens, F, kind="relu2", partials=None):
+    """out[t, f] = act(x[t, f]), x float32 rows or (partials) a product left in deferred mode."""
+    if kind not in UNIT_ACTS:
+        raise KernelError(f"unknown activation {kind!r}")
+    _need(out, None, "out", 2)
+    if partials is None:
+        _need(x, torch.float32, "x", 2)
+        _bytes_work((x, n_tokens), (out, n_tokens))
+    _check(lib().ferrum_unit_act(_ptr(x if partials is None else None), c_int(x.stride(0) if partials is None else 0), _ptr(out),
+                                 dtype_code(out.dtype), c_int(out.stride(0)), c_int(n_tokens), c_int(F),
+                                 _ptr(partials.workspace if partials is not None else None), partials._c if partials is not None else None,
+                                 _stream()), "unit_act")
 
 
 def rmsnorm(x, weight, out, eps, rows=None, n_rows=None, partials=None, groups=1):
@@ -414,7 +478,7 @@ def gemm_tc(x, w, out, epilogue, err, workspace, counters, M=None, N=None, dual_
     N = (w.shape[0] - dual_offset) if N is None else N
     if x.shape[1] != K or out.shape[1] < N or out.shape[0] < M or x.shape[0] < M:
         raise KernelError(f"gemm_tc: shapes do not agree: x {tuple(x.shape)} w {tuple(w.shape)} out {tuple(out.shape)}")
-    want = x.dtype if epilogue in (TC_STORE_BF16, TC_SWIGLU, TC_GEGLU, TC_SWISH_CLAMP) else torch.float32
+    want = x.dtype if epilogue in (TC_STORE_BF16, TC_SWIGLU, TC_GEGLU, TC_SWISH_CLAMP, TC_RELU2) else torch.float32
     if out.dtype != want:
         raise KernelError(f"gemm_tc: out must be {want} for epilogue {epilogue}")
     _need(workspace, torch.float32, "workspace")
@@ -714,7 +778,7 @@ def latent_prep(proj, n_tokens, off_q, q_rank, wq, off_kv, kv_rank, rot_dim, wkv
                                     c_int(off_kv), c_int(kv_rank), c_int(rot_dim), _ptr(wkv), c_int(off_gate), c_int(n_gate),
                                     _ptr(ctx.positions), _ptr(ctx.req_of_token), _ptr(block_table), c_int(block_table.shape[1]),
                                     _ptr(cos_sin), c_int(cos_sin.shape[0] if rot is not None else 0),
-                                    c_int(rot.rope_dim if rot is not None else 0), _ptr(plane if off_kv >= 0 else None),
+                                    c_int(rot.rope_dim if rot is not None else 0), c_int(rot.pairing if rot is not None else 0), _ptr(plane if off_kv >= 0 else None),
                                     c_longlong(page_stride), c_int(page_size), _ptr(cq), c_int(cq.stride(0)),
                                     dtype_code(cq.dtype), _ptr(gate), c_float(eps), _ptr(ctx.err),
                                     _ptr(partials.workspace if partials is not None else None),
@@ -728,7 +792,7 @@ def latent_q_rope(q, qf, n_tokens, positions, rot, H, Dn, Rr, R, err):
     _check(lib().ferrum_latent_q_rope(_ptr(q), c_int(q.stride(0)), _ptr(qf), c_int(qf.stride(0)), dtype_code(q.dtype),
                                       c_int(n_tokens), _ptr(positions), _ptr(cos_sin),
                                       c_int(cos_sin.shape[0] if rot is not None else 0),
-                                      c_int(rot.rope_dim if rot is not None else 0), c_int(H), c_int(Dn), c_int(Rr), c_int(R),
+                                      c_int(rot.rope_dim if rot is not None else 0), c_int(rot.pairing if rot is not None else 0), c_int(H), c_int(Dn), c_int(Rr), c_int(R),
                                       _ptr(err), _stream()), "latent_q_rope")
 
 
@@ -739,11 +803,13 @@ def attention_latent_split():
 
 
 def attention_latent(qf, out, gate, n_tokens, ctx, block_table, plane, page_stride, page_size, H, Dk, Dv, scale, window,
-                     single_tokens, part=None, split_slots=0, tensor_cores=None):
+                     single_tokens, part=None, split_slots=0, tensor_cores=None, sink=None, wide_weights=False):
     """Attention of every token over its request's cached rows of Dk elements, whose first Dv
     elements are the values; qf: heads of Dk, out: heads of Dv, times gate[t, h] (latent.cu).
     tensor_cores: None picks the mma.sync kernel where it takes the shape (16-bit storage, Dk a
     multiple of 16, Dv of 32), else the CUDA-core kernel; False forces the latter.
+    sink (float32 [H]): exp(sink[h]) joins the denominator of head h's softmax.  wide_weights: the tensor-core kernel
+    keeps the softmax weights to float32 precision (a 16-bit head and a 16-bit remainder) instead of rounding them.
     With `part` (float32, n_tokens * H * split_slots * (Dv + 2) elements; single tokens only) every
     token's keys are cut at multiples of `attention_latent_split()` among split_slots CTAs and folded
     by a second launch."""
@@ -762,17 +828,21 @@ def attention_latent(qf, out, gate, n_tokens, ctx, block_table, plane, page_stri
             _ptr(gate), c_int(n_tokens), _ptr(ctx.positions), _ptr(ctx.q_start), c_int(ctx.n_reqs),
             _ptr(block_table), c_int(block_table.shape[1]), _ptr(plane), c_longlong(page_stride),
             c_int(page_size), c_int(H), c_int(Dk), c_int(Dv), c_float(scale), c_int(window),
-            c_int(1 if single_tokens else 0), _ptr(part), c_int(split_slots), _ptr(ctx.err), _stream())
+            c_int(1 if single_tokens else 0), _ptr(part), c_int(split_slots), _ptr(sink), _ptr(ctx.err))
+    if sink is not None:
+        _need(sink, torch.float32, "sink", 1)
+        if sink.shape[0] != H or not sink.is_contiguous():
+            raise KernelError("attention_latent: one sink per head")
     if tensor_cores is None:
         tensor_cores = attention_latent_mma_supported(qf, out, plane, page_stride, Dk, Dv)
     if tensor_cores:
-        _check(lib().ferrum_attention_latent_mma(*args), "attention_latent_mma")
+        _check(lib().ferrum_attention_latent_mma(*args, c_int(1 if wide_weights else 0), _stream()), "attention_latent_mma")
         if part is not None:
             _check(lib().ferrum_attention_latent_combine(_ptr(out), c_int(out.stride(0)), dtype_code(out.dtype), _ptr(part), _ptr(gate),
                                                          c_int(n_tokens), _ptr(ctx.positions), c_int(H), c_int(Dv), c_int(window),
-                                                         c_int(split_slots), _stream()), "attention_latent_combine")
+                                                         c_int(split_slots), _ptr(sink), _stream()), "attention_latent_combine")
         return
-    _check(lib().ferrum_attention_latent(*args), "attention_latent")
+    _check(lib().ferrum_attention_latent(*args, _stream()), "attention_latent")
     if part is not None:
         globals()["launches"] += 1        # (the merge of the splits is a second kernel)
 
@@ -1044,12 +1114,14 @@ MOE_MAX_EXPERTS, MOE_MAX_TOP = 256, 8      # (the routing kernel's own limits, w
 
 
 def moe_route(logits, n_tokens, n_exp, top, x, scale_input, expert_of, rank_of, weight_of, counts, xg, row_of, scores="sigmoid",
-              renormalize=False, correction=None, weight_scale=1.0, n_identity=0, bias=None):
+              renormalize=False, correction=None, weight_scale=1.0, n_identity=0, bias=None, groups=None, renorm_eps=0.0):
     """From the router's float32 logits [T, >= n_exp]: every token's `top` experts and their weights, and the
     tokens' input rows x [T, E] gathered into xg [T * top, E] sorted by expert (times the weight when
     `scale_input`); row_of [T * top] says where each (token, choice) went; counts [n_exp] the rows per expert.
     bias (float32 [n_exp]) is added to the logits first.  correction (float32 [n_exp]) is added to the scores for the choice only; the weights are the plain scores times
-    weight_scale.  The last n_identity of the n_exp router outputs are identity experts: they get no rows (row_of -1)."""
+    weight_scale.  The last n_identity of the n_exp router outputs are identity experts: they get no rows (row_of -1).
+    groups = (count, keep): the experts form `count` equal groups of neighbours and only those of the `keep` best can be chosen, a
+    group being worth the sum of its two largest corrected scores.  renorm_eps is added to the sum that `renormalize` divides by."""
     global launches
     _need(logits, torch.float32, "logits", 2); _need(x, None, "x", 2); _need(xg, x.dtype, "xg", 2)
     for t in (expert_of, rank_of, counts, row_of):
@@ -1067,7 +1139,8 @@ def moe_route(logits, n_tokens, n_exp, top, x, scale_input, expert_of, rank_of, 
                                   c_int(MOE_SCORES[scores]), c_int(1 if renormalize else 0), _ptr(x), c_int(x.stride(0)), c_int(E),
                                   dtype_code(x.dtype), c_int(1 if scale_input else 0), _ptr(expert_of), _ptr(rank_of),
                                   _ptr(weight_of), _ptr(counts), _ptr(xg), _ptr(row_of), _ptr(correction), c_float(weight_scale),
-                                  c_int(n_identity), _ptr(bias), _stream()), "moe_route")
+                                  c_int(n_identity), _ptr(bias), c_int(groups[0] if groups else 0), c_int(groups[1] if groups else 0),
+                                  c_float(renorm_eps), _stream()), "moe_route")
     launches += 0 if n_tokens <= 16 and n_tokens * top <= 256 else 1          # (with many tokens: the routing and the gather)
 
 
@@ -1081,13 +1154,16 @@ def set_moe_tcgen05(on: bool):
     _moe_tcgen05 = bool(on)
 
 
-def moe_gemm(a, w, counts, n_rows, out, N, glu=None, err=None, limit=0.0):
+def moe_gemm(a, w, counts, n_rows, out, N, glu=None, err=None, limit=0.0, act=None):
     """out[row] = a[row] @ w[expert of row].T over rows sorted by expert (`counts` rows each, on the device).
     w: [n_exp, rows, K]; glu ("silu" / "gelu_tanh"): w holds N gate rows then N up rows per expert and out
-    (compute type) gets act(gate) * up; else out is float32 [n_rows, N].  With `err` (the step's error flag) 16-bit
+    (compute type) gets act(gate) * up; act ("relu2"): out (compute type) gets that activation of the product; else out is
+    float32 [n_rows, N].  With `err` (the step's error flag) 16-bit
     products of many rows (more than about 32 an expert) run on the tcgen05 kernel, the others on mma.sync tiles
     or, float32 and unaligned rows, on the CUDA cores."""
-    _need(a, None, "a", 2); _need(w, a.dtype, "w", 3); _need(out, a.dtype if glu else torch.float32, "out", 2)
+    _need(a, None, "a", 2); _need(w, a.dtype, "w", 3); _need(out, a.dtype if glu or act else torch.float32, "out", 2)
+    if act is not None and (glu or act not in UNIT_ACTS):
+        raise KernelError(f"moe_gemm: unknown activation {act!r} of an ungated unit")
     n_exp, w_rows, K = w.shape
     if not w.is_contiguous() or a.shape[1] != K or a.shape[0] < n_rows or out.shape[0] < n_rows or out.shape[1] < N:
         raise KernelError("moe_gemm: shapes do not agree")
@@ -1099,10 +1175,10 @@ def moe_gemm(a, w, counts, n_rows, out, N, glu=None, err=None, limit=0.0):
             and lib().ferrum_gemm_tc_grouped_supported(_ptr(a), _ptr(w), c_int(n_rows), c_int(n_exp), c_int(K), c_int(a.stride(0)))):
         _check(lib().ferrum_gemm_tc_grouped(_ptr(a), _ptr(w), _ptr(out), dtype_code(a.dtype), c_int(n_rows), c_int(a.shape[0]), c_int(N),
                                             c_int(K), c_int(a.stride(0)), c_int(out.stride(0)), c_int(n_exp), c_int(w_rows), _ptr(counts),
-                                            c_int(1 + GLU_ACTS[glu] if glu else 0), _ptr(err), c_float(limit), _stream()), "moe_gemm")
+                                            c_int(1 + GLU_ACTS[glu] if glu else (-1 if act else 0)), _ptr(err), c_float(limit), _stream()), "moe_gemm")
         return
     _check(lib().ferrum_moe_gemm(_ptr(a), c_int(a.stride(0)), _ptr(w), c_int(w_rows), c_int(K), c_int(N), c_int(n_exp), _ptr(counts),
-                                 c_int(n_rows), dtype_code(a.dtype), c_int(1 if glu else 0), c_int(GLU_ACTS[glu] if glu else 0), c_float(limit),
+                                 c_int(n_rows), dtype_code(a.dtype), c_int(1 if glu else 0), c_int(GLU_ACTS[glu] if glu else UNIT_ACTS[act] if act else 0), c_float(limit),
                                  _ptr(out), c_int(out.stride(0)), _stream()), "moe_gemm")
 
 

@@ -21,7 +21,7 @@ import torch
 
 from ..ops import lib as ops
 from .base import FeedForward, ParamSpec
-from .linear import RESIDUAL, STORE, STORE_F32, linear, linear_deferred, linear_swiglu
+from .linear import RESIDUAL, STORE, STORE_F32, linear, linear_deferred, linear_swiglu, linear_unit
 
 
 # Up to this many tokens in a step a routed feed-forward's unit for every token runs on a second stream beside the routing.
@@ -108,6 +108,33 @@ class SwiGLU(FeedForward):
         return None
 
 
+class PlainUnit(FeedForward):
+    """down(act(up(x))) without a gate, added to the residual stream.  On the tensor-core path the activation runs in the first
+    product's epilogue; in steps of a few tokens that product stays in partials, which the activation kernel sums; elsewhere
+    (float32, rows that are no 16-byte multiples) it leaves float32 rows, so that nothing is rounded before the activation."""
+    graph_safe = True
+
+    def __init__(self, width, hidden, dtype, act="relu2"):
+        if act not in ops.UNIT_ACTS:
+            raise ValueError(f"unknown activation {act!r}")
+        self.width, self.hidden, self.dtype, self.act = width, hidden, dtype, act
+        self.w_up_weight = self.w_down_weight = None
+
+    def param_specs(self):
+        return {"up.weight": ParamSpec((self.hidden, self.width)), "down.weight": ParamSpec((self.width, self.hidden))}
+
+    def forward(self, x, ctx, residual, accumulate=True, defer=False):
+        F, T = self.hidden, ctx.n_tokens
+        act = ctx.buf("unit_act", (ctx.token_capacity, F), self.dtype)
+        linear_unit(x, self.w_up_weight, act, ctx, T, self.act)
+        if defer and not accumulate:
+            part = linear_deferred(act, self.w_down_weight, ctx, T)
+            if part is not None:
+                return part
+        linear(act, self.w_down_weight, residual, RESIDUAL if accumulate else STORE_F32, ctx, M=T)
+        return None
+
+
 class RoutedFeedForward(FeedForward):
     """A mixture of experts: every token runs through `top` of `n_experts` small gated feed-forwards
     down_e(act(gate_e z) * (up_e z)), chosen by a router.
@@ -126,6 +153,12 @@ class RoutedFeedForward(FeedForward):
                     is the token's own input row, times the weight
     limit           the clamp of act "swish_clamp"
     shared          a `FeedForward` that every token runs through; its result joins the sum
+    gated           False: an expert is down_e(act(up_e z)), with an activation of `ops.UNIT_ACTS`
+    groups          (count, keep): the experts form `count` equal groups of neighbours, and only those of the `keep` best
+                    groups can be chosen; a group is worth the sum of its two largest (corrected) scores
+    renorm_eps      added to the sum that `renormalize` divides by
+    defer_sum       the sum into the residual rows may stay open for the norm that reads them next
+                    (StepContext.pending_experts)
 
     The tokens' rows are gathered into a buffer sorted by expert; two grouped products (gate/up with
     the activation, then down) run over it with the experts' stacked matrices, every CTA finding its
@@ -136,9 +169,16 @@ class RoutedFeedForward(FeedForward):
 
     def __init__(self, width, hidden, n_experts, top, dtype, act="silu", scores="sigmoid", renormalize=False, scale_input=True,
                  correction=False, weight_scale=1.0, identity=0, limit=0.0, shared: FeedForward = None,
-                 router_bias=False):
-        if act not in ops.GLU_ACTS:
+                 router_bias=False, gated=True, groups=None, renorm_eps=0.0, defer_sum=False):
+        if act not in (ops.GLU_ACTS if gated else ops.UNIT_ACTS):
             raise ValueError(f"unknown activation {act!r}")
+        self.gated, self.renorm_eps, self.defer_sum = bool(gated), float(renorm_eps), bool(defer_sum)
+        self.groups = None
+        if groups is not None:
+            count, keep = (int(v) for v in groups)
+            if identity or not (0 < keep <= count and n_experts % count == 0 and top <= n_experts // count * keep):
+                raise ValueError(f"{top} of {n_experts} experts cannot come from {keep} of {count} equal groups")
+            self.groups = (count, keep)
         if scores not in ops.MOE_SCORES:
             raise ValueError(f"unknown router scores {scores!r}")
         identity = int(identity)
@@ -164,8 +204,9 @@ class RoutedFeedForward(FeedForward):
         if self.has_correction:
             out["correction"] = ParamSpec((self.n_experts + self.identity,), kind="vector", init="normal")
         for e in range(self.n_experts):
-            out.update({f"e{e}.gate.weight": ParamSpec((self.hidden, self.width)),
-                        f"e{e}.up.weight": ParamSpec((self.hidden, self.width)),
+            if self.gated:
+                out[f"e{e}.gate.weight"] = ParamSpec((self.hidden, self.width))
+            out.update({f"e{e}.up.weight": ParamSpec((self.hidden, self.width)),
                         f"e{e}.down.weight": ParamSpec((self.width, self.hidden))})
         return out
 
@@ -179,8 +220,9 @@ class RoutedFeedForward(FeedForward):
             t = getattr(self, name)
             delattr(self, name)
             return t
-        gu = [torch.cat([take(f"w_e{e}_gate_weight"), take(f"w_e{e}_up_weight")], dim=0) for e in range(self.n_experts)]
-        self.w_gate_up = torch.stack(gu, dim=0).contiguous()                       # [experts, 2F, E]
+        gu = [torch.cat([take(f"w_e{e}_{k}_weight") for k in (("gate", "up") if self.gated else ("up",))], dim=0)
+              for e in range(self.n_experts)]
+        self.w_gate_up = torch.stack(gu, dim=0).contiguous()                       # [experts, 2F, E] (no gates: [experts, F, E])
         self.w_down = torch.stack([take(f"w_e{e}_down_weight") for e in range(self.n_experts)], dim=0).contiguous()   # [experts, E, F]
 
     def forward_rows(self, x, ctx):
@@ -198,9 +240,11 @@ class RoutedFeedForward(FeedForward):
         xg = ctx.buf("moe_x", (cap * top, self.width), self.dtype)
         ops.moe_route(logits, T, n_out, top, x, self.scale_input, expert_of, rank_of, weight_of, counts, xg, row_of,
                       scores=self.scores, renormalize=self.renormalize, correction=self.w_correction if self.has_correction else None,
-                      weight_scale=self.weight_scale, n_identity=self.identity, bias=self.w_router_bias if self.has_router_bias else None)
+                      weight_scale=self.weight_scale, n_identity=self.identity, bias=self.w_router_bias if self.has_router_bias else None,
+                      groups=self.groups, renorm_eps=self.renorm_eps)
         act = ctx.buf("moe_act", (cap * top, self.hidden), self.dtype)
-        ops.moe_gemm(xg, self.w_gate_up, counts, T * top, act, self.hidden, glu=self.act, err=ctx.err, limit=self.limit)
+        ops.moe_gemm(xg, self.w_gate_up, counts, T * top, act, self.hidden, glu=self.act if self.gated else None, err=ctx.err, limit=self.limit,
+                     act=None if self.gated else self.act)
         rows = ctx.buf("moe_rows", (cap * top, self.width), torch.float32)
         ops.moe_gemm(act, self.w_down, counts, T * top, rows, self.width, err=ctx.err)
         self._weight_of = weight_of
@@ -231,6 +275,10 @@ class RoutedFeedForward(FeedForward):
                 self.shared.forward(x, ctx, add, accumulate=False)
                 ctx.flush_residual()
         rows, row_of, top = self.forward_rows(x, ctx)
+        if self.defer_sum and accumulate and add is None and copy is None and not self.identity:
+            ctx.flush_residual()
+            ctx.pending_experts = (residual, ops.ExpertSum(rows, row_of, top, None if self.scale_input else self._weight_of))
+            return None
         if join is not None:
             torch.cuda.current_stream().wait_event(join)
         ops.moe_combine(rows, row_of, top, ctx.n_tokens, residual, weight_of=None if self.scale_input else self._weight_of,

@@ -8,7 +8,10 @@ out per head as [`dim` unrotated | `rot_dim` rotated], and the score of head h f
 (q' = [U_k,h^T q_plain | q_rot]) and the value map applied after the weighted sum, so attention
 runs on the cached rows themselves: one shared row of kv_rank + rot_dim key elements whose first
 kv_rank elements are the values, for all heads.  An output gate sigmoid(W_g x)_h scales head h
-before the output projection.  `window` > 0: a query at p sees keys p - window + 1 .. p.
+before the output projection.  `window` > 0: a query at p sees keys p - window + 1 .. p.  `rot_dim` 0: no rotated part (the
+score is the plain part's alone).  `sink`: exp(sink_h), a learned number per head, joins the denominator of head h's
+softmax; it has no value.  `wide_weights`: in 16-bit modes the softmax weights keep float32 precision also where the
+weighted sum runs on the tensor cores.
 
 A mixer built with `own_latent=False` has no down-projection for keys and values: it runs as a
 schedule entry with `cache_of`, reads the rows another run cached, and expands them with its own
@@ -36,18 +39,19 @@ class LatentAttention(Mixer):
     graph_safe = True
 
     def __init__(self, width, heads, dim, rot_dim, vdim, kv_rank, q_rank, eps, scale, dtype, rotary=None, window=0,
-                 own_latent=True):
-        """rotary: a `RotaryEmbedding` over the rot_dim part (its rope_dim leading elements turn,
-        "half" pairing), or None for no rotation."""
+                 own_latent=True, sink=False, wide_weights=False):
+        """rotary: a `RotaryEmbedding` over the rot_dim part (its rope_dim leading elements turn, in either pairing),
+        or None for no rotation."""
         self.width, self.H, self.Dn, self.Rr, self.Dv = width, int(heads), int(dim), int(rot_dim), int(vdim)
         self.R, self.Rq = int(kv_rank), int(q_rank)
         self.eps, self.scale, self.dtype = float(eps), float(scale), dtype
         self.rotary, self.window, self.own_latent = rotary, int(window), bool(own_latent)
-        if rotary is not None and (rotary.rope_dim > self.Rr or rotary.pairing != 1):
-            raise ValueError("the rotary table must cover at most rot_dim elements, paired (i, i + dims/2)")
+        self.has_sink, self.wide_weights = bool(sink), bool(wide_weights)
+        if rotary is not None and rotary.rope_dim > self.Rr:
+            raise ValueError("the rotary table must cover at most rot_dim elements")
         self.Dk = self.R + self.Rr
         for name in ("dq_weight", "dq_norm_weight", "uq_weight", "dkv_weight", "dkv_norm_weight", "uk_weight", "uv_weight",
-                     "g_weight", "o_weight"):
+                     "g_weight", "o_weight", "sink"):
             setattr(self, "w_" + name, None)
         self.w_in = self.w_uk_t = self.w_uv_h = None
 
@@ -57,6 +61,8 @@ class LatentAttention(Mixer):
                "uq.weight": ParamSpec((H * (self.Dn + self.Rr), self.Rq)),
                "uk.weight": ParamSpec((H * self.Dn, self.R)), "uv.weight": ParamSpec((H * self.Dv, self.R)),
                "g.weight": ParamSpec((H, E)), "o.weight": ParamSpec((E, H * self.Dv))}
+        if self.has_sink:
+            out["sink"] = ParamSpec((H,), kind="vector", init="normal")
         if self.own_latent:
             out["dkv.weight"] = ParamSpec((self.R + self.Rr, E))
             out["dkv_norm.weight"] = ParamSpec((self.R,), kind="vector", init="ones_normal")
@@ -121,7 +127,7 @@ class LatentAttention(Mixer):
             else:
                 slots = 0
         ops.attention_latent(qf, o, gate, T, ctx, table, cache.plane, cache.page_stride, cache.page_size, H, Dk, R,
-                             self.scale, self.window, single_tokens=single, part=part, split_slots=slots)
+                             self.scale, self.window, single_tokens=single, part=part, split_slots=slots, sink=self.w_sink, wide_weights=self.wide_weights)
         ov = ctx.buf("lat_ov", (cap, H * Dv), self.dtype)
         if few or ops.head_linear_mma_supported(o, R, self.w_uv_h, ov, Dv):
             ops.head_linear(o, R, self.w_uv_h, ov, Dv, T)

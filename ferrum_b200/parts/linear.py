@@ -52,6 +52,27 @@ def linear(x, w, out, mode, ctx, M=None):
         ops.gemm_generic(x, w, out, _GENERIC[mode], M=M)
 
 
+_UNIT_EPILOGUE = {"relu2": ops.TC_RELU2}
+
+
+def linear_unit(x, w, out, ctx, M, kind):
+    """out = act(x[:M] @ w.T) in the compute type, the activation applied to the unrounded product."""
+    if M == 0:
+        return
+    N, K = w.shape
+    part = linear_deferred(x, w, ctx, M) if ctx.defer_swiglu else None
+    if part is not None:
+        ops.unit_act(None, out, M, N, kind, partials=part)
+    elif ops.gemm_tc_supported(x, w):
+        ctx.flush_residual()
+        ws, cnt = ctx.gemm_scratch(M, N, K, False)
+        ops.gemm_tc(x, w, out, _UNIT_EPILOGUE[kind], ctx.err, ws, cnt, M=M)
+    else:
+        wide = ctx.buf("unit_wide", (ctx.token_capacity, N), torch.float32)
+        linear(x, w, wide, STORE_F32, ctx, M=M)
+        ops.unit_act(wide, out, M, N, kind)
+
+
 _GLU_EPILOGUE = {"silu": ops.TC_SWIGLU, "gelu_tanh": ops.TC_GEGLU, "swish_clamp": ops.TC_SWISH_CLAMP}
 
 

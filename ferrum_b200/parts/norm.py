@@ -4,6 +4,8 @@ mean square (the reference has one group).  `zero_centred`: the file stores the 
 the norm multiplies by 1 + w."""
 from __future__ import annotations
 
+import torch
+
 from ..ops import lib as ops
 from .base import Norm, ParamSpec
 
@@ -30,6 +32,8 @@ class RMSNorm(Norm):
         n = n_rows if n_rows is not None else ctx.n_tokens
         cap = ctx.want_capacity if rows is not None else ctx.token_capacity
         out = ctx.buf(tag + ("_rows" if rows is not None else ""), (cap, self.width), self.out_dtype)
+        if ctx.pending_experts is not None:
+            ctx.flush_residual()
         if self.groups > 1:
             ctx.flush_residual()
             ops.rmsnorm(h, self.w_weight, out, self.eps, rows=rows, n_rows=n, groups=self.groups)
@@ -44,4 +48,40 @@ class RMSNorm(Norm):
         elif ctx.pending_add is not None:
             ctx.flush_residual()
         ops.rmsnorm(h, self.w_weight, out, self.eps, rows=rows, n_rows=n, partials=ctx.take_pending_residual(h))
+        return out
+
+
+def _alpha_init(shape, g, device, std):
+    return 0.5 + 0.1 * torch.randn(shape, generator=g, device=device, dtype=torch.float32)
+
+
+class DynamicTanh(Norm):
+    """tanh(alpha * x) * w + b with a scalar alpha: no statistic of the row enters, so the kernel is elementwise and makes
+    whatever residual sum is still open on its way (a product left in partials, or a routed feed-forward's unsummed expert
+    rows).  `scale` multiplies the result (it is folded into w and b once, in float32): a model whose logits are scaled
+    by a constant gives it to its last norm, since the head is linear.  The reference's norm is `RMSNorm`'s."""
+    graph_safe = True
+
+    def __init__(self, width: int, out_dtype, scale: float = 1.0):
+        self.width, self.out_dtype, self.scale = width, out_dtype, float(scale)
+        self.w_weight = self.w_bias = self.w_alpha = None
+
+    def param_specs(self):
+        return {"weight": ParamSpec((self.width,), kind="vector", init="ones_normal"), "bias": ParamSpec((self.width,), kind="vector"),
+                "alpha": ParamSpec((), kind="vector", init=_alpha_init)}
+
+    def finalize(self):
+        self.w_alpha = self.w_alpha.reshape(1).contiguous()
+        if self.scale != 1.0:
+            self.w_weight, self.w_bias = self.w_weight * self.scale, self.w_bias * self.scale
+
+    def forward(self, h, ctx, rows=None, n_rows=None, tag="norm"):
+        n = n_rows if n_rows is not None else ctx.n_tokens
+        cap = ctx.want_capacity if rows is not None else ctx.token_capacity
+        out = ctx.buf(tag + ("_rows" if rows is not None else ""), (cap, self.width), self.out_dtype)
+        partials = ctx.take_pending_residual(h)
+        experts = ctx.take_pending_experts(h) if partials is None else None
+        if partials is None and experts is None:
+            ctx.flush_residual()
+        ops.dyn_tanh(h, self.w_alpha, self.w_weight, self.w_bias, out, rows=rows, n_rows=n, partials=partials, experts=experts)
         return out

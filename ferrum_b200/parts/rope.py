@@ -66,12 +66,27 @@ register_scaling("llama3", llama3_scaling)
 register_scaling("linear", linear_scaling)
 
 
+def yarn(rope_dim, theta, factor, original, fast, slow):
+    """(frequencies, magnitude) of the YaRN rule: pairs that turn at least `fast` times over `original` positions keep their
+    frequency, pairs that turn at most `slow` times have it divided by `factor`, and between the two pair indices (rounded
+    outwards, kept inside 0 .. rope_dim - 1) the two are blended linearly.  The magnitude, 0.1 ln(factor) + 1, multiplies
+    both cos and sin."""
+    def pair_index(turns):
+        return rope_dim * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))
+    first, last = max(math.floor(pair_index(fast)), 0), min(math.ceil(pair_index(slow)), rope_dim - 1)
+    out = []
+    for i, f in enumerate(inverse_frequencies(rope_dim, theta)):
+        ramp = min(max((i - first) / max(last - first, 0.001), 0.0), 1.0)
+        out.append(f / factor * ramp + f * (1.0 - ramp))
+    return out, 0.1 * math.log(factor) + 1.0
+
+
 class RotaryEmbedding(PositionEncoding):
     graph_safe = True
 
-    def __init__(self, head_dim, rope_dim, theta, scaling, pairing, max_positions, device, frequencies=None):
+    def __init__(self, head_dim, rope_dim, theta, scaling, pairing, max_positions, device, frequencies=None, magnitude=1.0):
         """frequencies: the R/2 rotation frequencies themselves, for a rule that is no function of
-        (theta, scaling block); theta and scaling are not looked at then."""
+        (theta, scaling block); theta and scaling are not looked at then.  magnitude: multiplies cos and sin."""
         if rope_dim % 2 or rope_dim > head_dim:
             raise ValueError("invalid rope dimension")
         self.head_dim, self.rope_dim = head_dim, rope_dim
@@ -83,7 +98,7 @@ class RotaryEmbedding(PositionEncoding):
             raise ValueError("a rotation of R dimensions needs R/2 frequencies")
         inv = torch.tensor(list(frequencies), dtype=torch.float64)
         ang = torch.arange(self.max_positions, dtype=torch.float64)[:, None] * inv[None, :]
-        table = torch.stack([torch.cos(ang), torch.sin(ang)], dim=-1).to(torch.float32)
+        table = (torch.stack([torch.cos(ang), torch.sin(ang)], dim=-1) * float(magnitude)).to(torch.float32)
         self.cos_sin = table.contiguous().to(device)      # [positions, rope_dim/2, 2]
 
     def rotary(self):
