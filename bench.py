@@ -3,7 +3,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
                     [--model llama31-8b|llama32-3b|llama2-7b] [--dtype bf16|fp16|fp32]
-                    [--workload decode|serve|latent|hybrid|streams|delta|decay] [--layers L] [--batch B] [--context S] [--trials N] [--size 2b|8b]
+                    [--workload decode|serve|latent|hybrid|streams|delta|decay|groups] [--layers L] [--batch B] [--context S] [--trials N] [--size 2b|8b]
 
 Prints ONE JSON line.
 
@@ -52,6 +52,12 @@ Vikupel of equal width, heads, layers and active feed-forward width.
 attention that keeps the first keys beside an RWKV-style recurrence; every layer with eight experts, three per token, and a
 per-layer token input; one pass of a loop around all layers) beside the closest of the other designs, a Pererax of equal
 width, heads, recurrent state, layers and feed-forward weights.
+
+`--workload groups`: the same comparison for the Lelutar design (dynamic-tanh norms, a table of token pairs; layers in turn:
+rotary attention + dense unit, latent attention without positions + experts, latent attention with a rotated part + experts,
+rotary attention + experts; eight experts in four groups of which two are kept, two per token; units without gates) beside
+the two closest of the other designs, a Zavesun (one stream, no window: its attention and its experts) and a Ruperax (its latent
+attention), both of equal width, heads, layers and feed-forward weights.
 
 Weights are random N(0, 0.02); token ids are uniform random from a seed.  No L2 flush is needed
 between steps: a step reads gigabytes of weights, far more than the 126 MB L2 holds.
@@ -198,8 +204,8 @@ def main():
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the model has (named in config)")
     ap.add_argument("--model", default="llama31-8b", choices=sorted(MODELS), help="layer sizes (random weights)")
     ap.add_argument("--dtype", default="bf16", choices=sorted(DTYPES), help="compute dtype; fp32 is the true 32-bit path")
-    ap.add_argument("--workload", default="decode", choices=["decode", "serve", "latent", "hybrid", "streams", "delta", "decay"])
-    ap.add_argument("--size", default="2b", choices=sorted(LATENT_SIZES), help="latent, hybrid, streams, delta, decay: the layer sizes to compare at")
+    ap.add_argument("--workload", default="decode", choices=["decode", "serve", "latent", "hybrid", "streams", "delta", "decay", "groups"])
+    ap.add_argument("--size", default="2b", choices=sorted(LATENT_SIZES), help="latent, hybrid, streams, delta, decay, groups: the layer sizes to compare at")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--context", type=int, default=None,
                     help="cached tokens per request of the headline point (default 8192 for llama31-8b, 4096 for "
@@ -228,6 +234,8 @@ def main():
         return latent(args, design="pererax")
     if args.workload == "decay":
         return latent(args, design="tikunex")
+    if args.workload == "groups":
+        return latent(args, design="lelutar")
     return decode(args)
 
 
@@ -648,11 +656,42 @@ def decay_configs(size, layers, vocab=32000, window=1024):
     return ours, delta_configs(size, layers, vocab, window)[0]
 
 
+# Lelutar at the same two widths: attention and latent attention as in the Zavesun and the Ruperax above; a unit without a gate
+# has two matrices instead of three, so it is half as wide again for equal weights.
+GROUP_SIZES = {
+    "2b": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, rot_dim=64, kv_rank=512, q_rank=768, ff=8448, experts=8, top=2, groups=4, keep=2,
+               expert_ff=4224),
+    "8b": dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=128, rot_dim=64, kv_rank=512, q_rank=1536, ff=21504, experts=8, top=2, groups=4, keep=2,
+               expert_ff=10752),
+}
+
+
+def group_configs(size, layers, vocab=32000, window=4096):
+    """Layers in turn: attention + dense, latent + experts, rotated latent + experts, attention + experts; and a Zavesun and a
+    Ruperax of equal size beside it (`window` is wider than the runs are long: everybody sees every key)."""
+    s = GROUP_SIZES[size]
+    yarn = {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+    att = {"type": "attention", "mixer": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["vdim"], "scale": s["dim"] ** -0.5,
+                                          "rot": {"base": 50000.0, "dims": s["dim"], "scaling": yarn}}}
+    lat = {"heads": s["heads"], "dim": s["dim"], "vdim": s["vdim"], "kv_rank": s["kv_rank"], "q_rank": s["q_rank"], "scale": s["dim"] ** -0.5}
+    turned = dict(lat, rot_dim=s["rot_dim"], scale=(s["dim"] + s["rot_dim"]) ** -0.5, rot={"base": 50000.0, "dims": s["rot_dim"], "scaling": yarn})
+    dense = {"kind": "dense", "ff": s["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": s["expert_ff"]},
+           "router": {"experts": s["experts"], "top": s["top"], "groups": {"count": s["groups"], "keep": s["keep"]}}}
+    kinds = [dict(att, mlp=dense), {"type": "latent_attention", "mixer": lat, "mlp": moe}, {"type": "latent_attention_2", "mixer": turned, "mlp": moe},
+             dict(att, mlp=moe)]
+    ours = {"architecture": "Lelutar", "vocab": vocab, "width": s["width"], "norm": {"eps": 1e-6}, "logit_scale": 0.7,
+            "embedding": {"scale": 4.0, "bigram": {"buckets": vocab, "mul_prev": 31337, "mul_cur": 271}}, "layers": [kinds[i % 4] for i in range(layers)]}
+    zavesun = dict(stream_configs(size, layers, vocab, window)[0], streams=1)
+    return ours, zavesun, latent_configs(size, layers, vocab, window)[0]
+
+
 # design -> (title, configs of the design and of the model beside it, sizes, window, what stands beside it)
 DESIGNS = {"ruperax": ("Ruperax", latent_configs, LATENT_SIZES, 4096, "llama"), "vikupel": ("Vikupel", hybrid_configs, HYBRID_SIZES, 1024, "llama"),
            "zavesun": ("Zavesun", stream_configs, STREAM_SIZES, 1024, "llama"),
            "pererax": ("Pererax", delta_configs, DELTA_SIZES, 1024, "vikupel"),
-           "tikunex": ("Tikunex", decay_configs, DECAY_SIZES, 1024, "pererax")}
+           "tikunex": ("Tikunex", decay_configs, DECAY_SIZES, 1024, "pererax"),
+           "lelutar": ("Lelutar", group_configs, GROUP_SIZES, 0, ("zavesun", "ruperax"))}
 
 
 def latent(args, design="ruperax"):
@@ -680,7 +719,8 @@ def latent(args, design="ruperax"):
     with ClockSampler() as clk:
         title, make_configs, all_sizes, window, beside = DESIGNS[design]
         configs = make_configs(args.size, L)
-        for name, cfgd in zip((design, beside), configs):
+        beside = (beside,) if isinstance(beside, str) else beside
+        for name, cfgd in zip((design, *beside), configs):
             arch = registry.lookup(registry.architecture_name(cfgd))
             cfg = arch.read_config(cfgd)
             model = arch.build(cfg, td, "cuda", max_positions=max_len)
@@ -764,7 +804,7 @@ def latent(args, design="ruperax"):
                            vocab=32000, page_size=page,
                            parallelism="single GPU", l2="weights of a step exceed the L2 at these sizes"),
             "clocks": clk.summary(), "gpu_launches": int(ours["decode_launches_per_step"] * K), "peaks": pk,
-            design: ours, beside + "_equal_size": out[beside]}
+            design: ours, **{b + "_equal_size": out[b] for b in beside}}
     print(json.dumps(line))
     return 0
 

@@ -35,6 +35,10 @@ SPLIT_BELOW = 4
 MAX_SPLITS = 1024       # what the merge kernel folds per (token, head)
 
 
+def _sink_init(shape, g, device, std):
+    return torch.randn(shape, generator=g, device=device, dtype=torch.float32)
+
+
 class LatentAttention(Mixer):
     graph_safe = True
 
@@ -62,7 +66,7 @@ class LatentAttention(Mixer):
                "uk.weight": ParamSpec((H * self.Dn, self.R)), "uv.weight": ParamSpec((H * self.Dv, self.R)),
                "g.weight": ParamSpec((H, E)), "o.weight": ParamSpec((E, H * self.Dv))}
         if self.has_sink:
-            out["sink"] = ParamSpec((H,), kind="vector", init="normal")
+            out["sink"] = ParamSpec((H,), kind="vector", init=_sink_init)
         if self.own_latent:
             out["dkv.weight"] = ParamSpec((self.R + self.Rr, E))
             out["dkv_norm.weight"] = ParamSpec((self.R,), kind="vector", init="ones_normal")
