@@ -15,6 +15,9 @@
 // output; otherwise it writes (m, l, O) partials and `attention_combine` merges the
 // splits in a fixed order.
 //
+// WIDE: the softmax weights keep float32 precision on their way into the matrix unit.  A weight goes in as its rounding to
+// the 16-bit type and as the rounding of what that leaves out; both products go to the same float32 accumulators.
+//
 // Two ways to hand out work.  Grid (items, Hkv): one item per CTA and KV head (prompt
 // portions).  Or a balanced list: the host cuts the line of all (request, KV head, 64-key
 // tile) units into one equal share per CTA slot of the GPU; a share is a few items, each
@@ -83,6 +86,11 @@ __device__ __forceinline__ unsigned pack16(float lo, float hi) {
   return HALF ? pack2<__half>(lo, hi) : pack2<__nv_bfloat16>(lo, hi);
 }
 
+template <bool HALF>
+__device__ __forceinline__ float unpack16(unsigned bits) {
+  return HALF ? __half2float(__ushort_as_half((unsigned short)bits)) : __uint_as_float(bits << 16);
+}
+
 // element (row, col) of a [rows][D] 16-bit tile whose 16-byte chunks are XOR-swizzled by row
 template <int D>
 __device__ __forceinline__ elem16* tile_ptr(elem16* base, int row, int col) {
@@ -90,7 +98,7 @@ __device__ __forceinline__ elem16* tile_ptr(elem16* base, int row, int col) {
   return base + row * D + (chunk << 3) + (col & 7);
 }
 
-template <int D, int WM, int WN, bool HALF>
+template <int D, int WM, int WN, bool HALF, bool WIDE>
 __device__ __forceinline__ void flash_item(const FlashParams& p, const int* wk, int kvh, uint8_t* smem_raw) {
   constexpr int BM = 16 * WM;
   constexpr int NT = WM * WN * 32;
@@ -274,6 +282,14 @@ __device__ __forceinline__ void flash_item(const FlashParams& p, const int* wk, 
       a[1] = pack16<HALF>(s[2 * ks][2], s[2 * ks][3]);
       a[2] = pack16<HALF>(s[2 * ks + 1][0], s[2 * ks + 1][1]);
       a[3] = pack16<HALF>(s[2 * ks + 1][2], s[2 * ks + 1][3]);
+      unsigned rest[WIDE ? 4 : 1];
+      if constexpr (WIDE) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float* v = &s[2 * ks + (i >> 1)][(i & 1) * 2];
+          rest[i] = pack16<HALF>(v[0] - unpack16<HALF>(a[i] & 0xFFFFu), v[1] - unpack16<HALF>(a[i] >> 16));
+        }
+      }
 #pragma unroll
       for (int db = 0; db < D / 16; ++db) {
         unsigned b[4];
@@ -281,6 +297,10 @@ __device__ __forceinline__ void flash_item(const FlashParams& p, const int* wk, 
         ldmatrix_x4_trans(b, tile_ptr<D>(tV, r, db * 16 + (lane >> 4) * 8));
         mma16<HALF>(o[2 * db], a, b[0], b[1]);
         mma16<HALF>(o[2 * db + 1], a, b[2], b[3]);
+        if constexpr (WIDE) {
+          mma16<HALF>(o[2 * db], rest, b[0], b[1]);
+          mma16<HALF>(o[2 * db + 1], rest, b[2], b[3]);
+        }
       }
     }
     __syncthreads();  // everyone is done with this buffer before the next load overwrites it
@@ -346,7 +366,7 @@ __device__ __forceinline__ void flash_item(const FlashParams& p, const int* wk, 
   }
 }
 
-template <int D, int WM, int WN, bool HALF>
+template <int D, int WM, int WN, bool HALF, bool WIDE>
 __global__ void __launch_bounds__(WM * WN * 32)
 flash_kernel(const FlashParams p) {
   extern __shared__ __align__(128) uint8_t smem_raw[];
@@ -366,14 +386,14 @@ flash_kernel(const FlashParams p) {
 #pragma unroll
     for (int i = 0; i < 8; ++i) item[i] = wk[i];
     item[5] = item[5] * p.Hkv + blockIdx.y;
-    flash_item<D, WM, WN, HALF>(p, item, blockIdx.y, smem_raw);
+    flash_item<D, WM, WN, HALF, WIDE>(p, item, blockIdx.y, smem_raw);
     TRACE_MARK(TRACE_EXIT);
     return;
   }
   const int begin = p.cta_items[blockIdx.x], end = p.cta_items[blockIdx.x + 1];
   for (int w = begin; w < end; ++w) {
     const int* wk = p.work + (size_t)w * 8;
-    flash_item<D, WM, WN, HALF>(p, wk, wk[6], smem_raw);
+    flash_item<D, WM, WN, HALF, WIDE>(p, wk, wk[6], smem_raw);
     __syncthreads();  // the next item's loads reuse the shared memory the merge just read
   }
   TRACE_MARK(TRACE_EXIT);
@@ -475,22 +495,27 @@ combine_kernel(elem16* out, int ldo, const float* part_o, const float* part_ml, 
   *reinterpret_cast<uint2*>(out + (size_t)t * ldo + (size_t)head * D + d) = packed;
 }
 
-template <int D, int WM, int WN, bool HALF>
-int launch_flash(const FlashParams& p, int n_work, int n_ctas, cudaStream_t stream) {
+template <int D, int WM, int WN, bool HALF, bool WIDE>
+int launch_flash_as(const FlashParams& p, int n_work, int n_ctas, cudaStream_t stream) {
   constexpr int BM = 16 * WM;
   constexpr int kv_bytes = 4 * BN * D * 2 + BM * D * 2;
   constexpr int merge_bytes = WN * BM * (D + 2) * 4;
   constexpr int smem = kv_bytes > merge_bytes ? kv_bytes : merge_bytes;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(flash_kernel<D, WM, WN, HALF>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(flash_kernel<D, WM, WN, HALF, WIDE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     FERRUM_CHECK_ARG(e == cudaSuccess, "attention_flash: cannot reserve %d bytes of shared memory: %s", smem, cudaGetErrorString(e));
     configured = true;
   }
   dim3 grid = p.cta_items ? dim3(n_ctas, 1) : dim3(n_work, p.Hkv);
-  launch_kernel(flash_kernel<D, WM, WN, HALF>, grid, dim3(WM * WN * 32), smem, stream, p);
+  launch_kernel(flash_kernel<D, WM, WN, HALF, WIDE>, grid, dim3(WM * WN * 32), smem, stream, p);
   FERRUM_CHECK_LAUNCH("attention_flash");
   return 0;
+}
+
+template <int D, int WM, int WN, bool HALF>
+int launch_flash(const FlashParams& p, int n_work, int n_ctas, int wide, cudaStream_t stream) {
+  return wide ? launch_flash_as<D, WM, WN, HALF, true>(p, n_work, n_ctas, stream) : launch_flash_as<D, WM, WN, HALF, false>(p, n_work, n_ctas, stream);
 }
 
 }  // namespace
@@ -506,7 +531,7 @@ FERRUM_API int ferrum_attention_flash(const void* q, int ldq, void* out, int ldo
                                       long long page_stride, int page_size, const int* block_table, int table_width,
                                       const int* q_start, const int* pos0, const int* work, int n_work,
                                       const int* cta_items, int n_ctas, float* part_o, float* part_ml, int Hq, int Hkv,
-                                      int D, float scale, int window, int bm, int trigger_early, int* err_flag,
+                                      int D, float scale, int window, int bm, int trigger_early, int* err_flag, int wide,
                                       cudaStream_t stream) {
   FERRUM_CHECK_ARG(Hq > 0 && Hkv > 0 && Hq % Hkv == 0, "attention_flash: bad head counts Hq=%d Hkv=%d", Hq, Hkv);
   FERRUM_CHECK_ARG(ferrum_is_16bit(dtype), "attention_flash: dtype code %d is not a 16-bit type", dtype);
@@ -532,15 +557,15 @@ FERRUM_API int ferrum_attention_flash(const void* q, int ldq, void* out, int ldo
   p.trigger_early = trigger_early;
   p.scale_log2 = scale * 1.4426950408889634f;
   if (dtype == FERRUM_F16) {
-    if (D == 64 && bm == 16) return launch_flash<64, 1, 4, true>(p, n_work, n_ctas, stream);
-    if (D == 64 && bm == 64) return launch_flash<64, 4, 1, true>(p, n_work, n_ctas, stream);
-    if (D == 128 && bm == 16) return launch_flash<128, 1, 4, true>(p, n_work, n_ctas, stream);
-    return launch_flash<128, 4, 1, true>(p, n_work, n_ctas, stream);
+    if (D == 64 && bm == 16) return launch_flash<64, 1, 4, true>(p, n_work, n_ctas, wide, stream);
+    if (D == 64 && bm == 64) return launch_flash<64, 4, 1, true>(p, n_work, n_ctas, wide, stream);
+    if (D == 128 && bm == 16) return launch_flash<128, 1, 4, true>(p, n_work, n_ctas, wide, stream);
+    return launch_flash<128, 4, 1, true>(p, n_work, n_ctas, wide, stream);
   }
-  if (D == 64 && bm == 16) return launch_flash<64, 1, 4, false>(p, n_work, n_ctas, stream);
-  if (D == 64 && bm == 64) return launch_flash<64, 4, 1, false>(p, n_work, n_ctas, stream);
-  if (D == 128 && bm == 16) return launch_flash<128, 1, 4, false>(p, n_work, n_ctas, stream);
-  return launch_flash<128, 4, 1, false>(p, n_work, n_ctas, stream);
+  if (D == 64 && bm == 16) return launch_flash<64, 1, 4, false>(p, n_work, n_ctas, wide, stream);
+  if (D == 64 && bm == 64) return launch_flash<64, 4, 1, false>(p, n_work, n_ctas, wide, stream);
+  if (D == 128 && bm == 16) return launch_flash<128, 1, 4, false>(p, n_work, n_ctas, wide, stream);
+  return launch_flash<128, 4, 1, false>(p, n_work, n_ctas, wide, stream);
 }
 
 FERRUM_API int ferrum_attention_combine(void* out, int ldo, int dtype, const float* part_o, const float* part_ml,

@@ -15,6 +15,8 @@
 // P never passes through shared memory: the matrix unit fetches its shared-memory operands at
 // about 64 bytes a cycle, and with Q re-read for every 64 keys that fetch, not the arithmetic,
 // is what a stage costs (16 x 6 KB for the scores, 8 x 4 KB for the values).
+// WIDE keeps the softmax weights to float32 precision: what the rounding to 16 bits leaves out of P is rounded too and
+// stored over the second half of the scores' columns, and P V gets four more steps with that half as its operand.
 // S has two buffers per row tile, so the matrix unit computes the scores of the stage after next
 // while the threads of a tile work on P: a tile's threads never wait for a product that
 // depends on their own P, and the two tiles share the matrix unit.  The running maximum is only moved (and O rescaled, in tensor
@@ -172,7 +174,12 @@ __device__ __forceinline__ uint32_t pack2_16(float lo, float hi) {
   return HALF ? pack2<__half>(lo, hi) : pack2<__nv_bfloat16>(lo, hi);
 }
 
-template <int D, int NT, int BN, int NS, bool HALF>
+template <bool HALF>
+__device__ __forceinline__ float unpack_16(uint32_t bits) {
+  return HALF ? __half2float(__ushort_as_half((unsigned short)bits)) : __uint_as_float(bits << 16);
+}
+
+template <int D, int NT, int BN, int NS, bool HALF, bool WIDE>
 __global__ void __launch_bounds__(AttnTcConfig<D, NT, BN, NS>::THREADS, 1)
 attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, const AttnTcParams p) {
   using Cfg = AttnTcConfig<D, NT, BN, NS>;
@@ -329,6 +336,11 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         for (int kk = 0; kk < BN / 16; ++kk)  // 16 keys on: 8 columns of P, 16 rows of V
           umma_bf16_ts(o_tmem, p_tmem + kk * 8, umma_desc_mn_sw128(v_addr + kk * 16 * 128, Cfg::KV_HALF_BYTES, 1024), idesc_pv,
                        accumulate || kk > 0);
+        if constexpr (WIDE) {
+#pragma unroll
+          for (int kk = 0; kk < BN / 16; ++kk)  // the remainders, behind P
+            umma_bf16_ts(o_tmem, p_tmem + BN / 2 + kk * 8, umma_desc_mn_sw128(v_addr + kk * 16 * 128, Cfg::KV_HALF_BYTES, 1024), idesc_pv, true);
+        }
       };
       // the scores of stages 0 and 1 go ahead; in the loop the scores of stage j + 2 follow P V of stage j
       bool ok = mbar_wait(q_full, 0, abort_p);
@@ -468,6 +480,12 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         l3 += e3;
         pk[c / 2] = pack2_16<HALF>(e0, e1);
         pk[c / 2 + 1] = pack2_16<HALF>(e2, e3);
+        if constexpr (WIDE) {      // (the scores are done with: their registers keep what the rounding left out)
+          s[c] = e0 - unpack_16<HALF>(pk[c / 2] & 0xFFFFu);
+          s[c + 1] = e1 - unpack_16<HALF>(pk[c / 2] >> 16);
+          s[c + 2] = e2 - unpack_16<HALF>(pk[c / 2 + 1] & 0xFFFFu);
+          s[c + 3] = e3 - unpack_16<HALF>(pk[c / 2 + 1] >> 16);
+        }
       }
       l_run += (l0 + l1) + (l2 + l3);
       if (j + 1 == n_j && kv_end - key0 < BN) {
@@ -496,6 +514,12 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       // measured slower: the wait is not what a stage spends its time on.)
 #pragma unroll
       for (int c0 = 0; c0 < BN / 2; c0 += 32) tmem_st32u(lane_addr + Cfg::S_COL + (2 * t + buf) * BN + c0, &pk[c0]);
+      if constexpr (WIDE) {
+#pragma unroll
+        for (int c = 0; c < BN; c += 2) pk[c / 2] = pack2_16<HALF>(s[c], s[c + 1]);
+#pragma unroll
+        for (int c0 = 0; c0 < BN / 2; c0 += 32) tmem_st32u(lane_addr + Cfg::S_COL + (2 * t + buf) * BN + BN / 2 + c0, &pk[c0]);
+      }
       tc_fence_before();     // this thread's tensor-memory accesses precede the products that follow
       // A warp may be a stage ahead of the tile's other warps (the next scores do not wait for
       // this P), so odd and even stages announce P on barriers of their own: an arrival is never
@@ -1080,18 +1104,24 @@ int cache_map(const void* plane, long long n_pages, int Hkv, int page_size, int 
   return 0;
 }
 
-template <int D, int NT, int BN, int NS, bool HALF>
-int launch_attention_tc(const CUtensorMap& mq, const CUtensorMap& mkv, const AttnTcParams& p, int n_work, cudaStream_t stream) {
+template <int D, int NT, int BN, int NS, bool HALF, bool WIDE>
+int launch_attention_tc_as(const CUtensorMap& mq, const CUtensorMap& mkv, const AttnTcParams& p, int n_work, cudaStream_t stream) {
   using Cfg = AttnTcConfig<D, NT, BN, NS>;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel<D, NT, BN, NS, HALF>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES);
+    cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel<D, NT, BN, NS, HALF, WIDE>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES);
     FERRUM_CHECK_ARG(e == cudaSuccess, "attention_tc: cannot reserve %d bytes of shared memory: %s", Cfg::SMEM_BYTES, cudaGetErrorString(e));
     configured = true;
   }
-  launch_kernel(attention_tc_kernel<D, NT, BN, NS, HALF>, dim3(p.Hkv, n_work), dim3(Cfg::THREADS), Cfg::SMEM_BYTES, stream, mq, mkv, p);
+  launch_kernel(attention_tc_kernel<D, NT, BN, NS, HALF, WIDE>, dim3(p.Hkv, n_work), dim3(Cfg::THREADS), Cfg::SMEM_BYTES, stream, mq, mkv, p);
   FERRUM_CHECK_LAUNCH("attention_tc");
   return 0;
+}
+
+template <int D, int NT, int BN, int NS, bool HALF>
+int launch_attention_tc(const CUtensorMap& mq, const CUtensorMap& mkv, const AttnTcParams& p, int n_work, int wide, cudaStream_t stream) {
+  return wide ? launch_attention_tc_as<D, NT, BN, NS, HALF, true>(mq, mkv, p, n_work, stream)
+              : launch_attention_tc_as<D, NT, BN, NS, HALF, false>(mq, mkv, p, n_work, stream);
 }
 
 template <int NS, bool HALF>
@@ -1153,7 +1183,7 @@ FERRUM_API int ferrum_attention_tc(const void* q, int ldq, long long q_rows, voi
                                    long long page_stride, long long n_pages, int page_size, const int* block_table,
                                    int table_width, const int* q_start, const int* pos0, const int* work, int n_work,
                                    float* part_o, float* part_ml, int Hq, int Hkv, int D, float scale, int window,
-                                   int* err_flag, cudaStream_t stream) {
+                                   int* err_flag, int wide, cudaStream_t stream) {
   FERRUM_CHECK_ARG(Hq > 0 && Hkv > 0 && Hq % Hkv == 0, "attention_tc: bad head counts Hq=%d Hkv=%d", Hq, Hkv);
   const int G = Hq / Hkv;
   const int tok = ferrum_attention_tc_tokens(D, G, page_size) / TC_TILES;
@@ -1179,15 +1209,15 @@ FERRUM_API int ferrum_attention_tc(const void* q, int ldq, long long q_rows, voi
   p.scale_log2 = scale * 1.4426950408889634f;
   CUtensorMap mq, mkv;
   if (int r = cache_map(kv_plane, n_pages, Hkv, page_size, D, &mkv)) return r;
-  if (D == 128 && g_attention_pair) {
+  if (D == 128 && g_attention_pair && !wide) {
     if (dtype == FERRUM_F16) return launch_attention_tc_pair<3, true>(mkv, q, ldq, p, n_work, stream);
     return launch_attention_tc_pair<3, false>(mkv, q, ldq, p, n_work, stream);
   }
   if (int r = query_map(q, q_rows, ldq, Hq, D, G, tok, &mq)) return r;
   if (dtype == FERRUM_F16) {
-    if (D == 64) return launch_attention_tc<64, TC_TILES, TC_BN, TC_STAGES, true>(mq, mkv, p, n_work, stream);
-    return launch_attention_tc<128, TC_TILES, TC_BN, TC_STAGES, true>(mq, mkv, p, n_work, stream);
+    if (D == 64) return launch_attention_tc<64, TC_TILES, TC_BN, TC_STAGES, true>(mq, mkv, p, n_work, wide, stream);
+    return launch_attention_tc<128, TC_TILES, TC_BN, TC_STAGES, true>(mq, mkv, p, n_work, wide, stream);
   }
-  if (D == 64) return launch_attention_tc<64, TC_TILES, TC_BN, TC_STAGES, false>(mq, mkv, p, n_work, stream);
-  return launch_attention_tc<128, TC_TILES, TC_BN, TC_STAGES, false>(mq, mkv, p, n_work, stream);
+  if (D == 64) return launch_attention_tc<64, TC_TILES, TC_BN, TC_STAGES, false>(mq, mkv, p, n_work, wide, stream);
+  return launch_attention_tc<128, TC_TILES, TC_BN, TC_STAGES, false>(mq, mkv, p, n_work, wide, stream);
 }

@@ -49,7 +49,8 @@ def build_lelutar(config: LelutarConfig, dtype, device, max_positions=None):
     for i in c.owners():
         m, p = c.layers[i].mixer, c.layers[i].mlp
         if isinstance(m, AttentionSpec):
-            mixer = ShapedAttention(E, m.heads, m.kv_heads, m.dim, m.vdim, dtype, m.scale, rotary=rotary(m.dim, m.rot), qkv_bias=True)
+            mixer = ShapedAttention(E, m.heads, m.kv_heads, m.dim, m.vdim, dtype, m.scale, rotary=rotary(m.dim, m.rot), qkv_bias=True,
+                                    wide_weights=True)
         else:
             mixer = LatentAttention(E, m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank, m.q_rank, c.norm_eps, m.scale, dtype,
                                     rotary=rotary(m.rot_dim, m.rot), sink=True, wide_weights=True)

@@ -26,7 +26,7 @@ TC_STORE_BF16, TC_STORE_F32, TC_RESIDUAL, TC_SWIGLU, TC_GEGLU, TC_SWISH_CLAMP, T
 
 _lib = None
 _lock = threading.Lock()
-ABI = 19
+ABI = 21
 
 
 def lib():
@@ -606,9 +606,10 @@ def profiling():
 
 
 def attention_flash(q, out, kv_plane, page_stride, page_size, block_table, q_start, pos0, work, n_work, part_o,
-                    part_ml, Hq, Hkv, D, scale, window, bm, err, cta_items=None, n_ctas=0, trigger_early=False):
+                    part_ml, Hq, Hkv, D, scale, window, bm, err, cta_items=None, n_ctas=0, trigger_early=False, wide_weights=False):
     """Tensor-core attention over the work items of one row-tile class (bm 16 or 64).
-    trigger_early: the kernels that follow in the stream may start while this one runs."""
+    trigger_early: the kernels that follow in the stream may start while this one runs.  wide_weights: the softmax weights
+    keep float32 precision (a 16-bit head and a 16-bit remainder) instead of being rounded for the second product."""
     _need16(q, "q", 2); _need16(out, "out", 2, like=q); _need16(kv_plane, "kv_plane", like=q)
     _need(block_table, torch.int32, "block_table", 2); _need(work, torch.int32, "work", 1)
     _check(lib().ferrum_attention_flash(_ptr(q), c_int(q.stride(0)), _ptr(out), c_int(out.stride(0)), dtype_code(q.dtype),
@@ -618,7 +619,7 @@ def attention_flash(q, out, kv_plane, page_stride, page_size, block_table, q_sta
                                         c_int(n_work), _ptr(cta_items), c_int(n_ctas), _ptr(part_o), _ptr(part_ml),
                                         c_int(Hq), c_int(Hkv), c_int(D),
                                         c_float(scale), c_int(window), c_int(bm), c_int(1 if trigger_early else 0),
-                                        _ptr(err), _stream()), "attention_flash")
+                                        _ptr(err), c_int(1 if wide_weights else 0), _stream()), "attention_flash")
 
 
 def attention_tc_tokens(D, G, page_size, kv_plane=None, page_stride=0):
@@ -638,15 +639,15 @@ def set_attention_pair_kernel(on: bool):
 
 
 def attention_tc(q, out, kv_plane, page_stride, page_size, block_table, q_start, pos0, work, n_work, part_o, part_ml,
-                 Hq, Hkv, D, scale, window, err):
-    """tcgen05 attention over work items of attention_tc_tokens * G rows (prompt portions)."""
+                 Hq, Hkv, D, scale, window, err, wide_weights=False):
+    """tcgen05 attention over work items of attention_tc_tokens * G rows (prompt portions).  wide_weights: as in `attention_flash`."""
     _need16(q, "q", 2); _need16(out, "out", 2, like=q); _need16(kv_plane, "kv_plane", like=q)
     _need(block_table, torch.int32, "block_table", 2); _need(work, torch.int32, "work", 1)
     _check(lib().ferrum_attention_tc(_ptr(q), c_int(q.stride(0)), c_longlong(q.shape[0]), _ptr(out), c_int(out.stride(0)),
                                      dtype_code(q.dtype), _ptr(kv_plane), c_longlong(page_stride), c_longlong(kv_plane.shape[0]),
                                      c_int(page_size), _ptr(block_table), c_int(block_table.shape[1]), _ptr(q_start),
                                      _ptr(pos0), _ptr(work), c_int(n_work), _ptr(part_o), _ptr(part_ml), c_int(Hq),
-                                     c_int(Hkv), c_int(D), c_float(scale), c_int(window), _ptr(err), _stream()),
+                                     c_int(Hkv), c_int(D), c_float(scale), c_int(window), _ptr(err), c_int(1 if wide_weights else 0), _stream()),
            "attention_tc")
 
 

@@ -49,6 +49,7 @@ class PagedAttention(Mixer):
         self.chunked = False     # True: `window` is a chunk length (a subclass sets it)
         self.keep_first = 0      # with a window: the sequence's first keys that every query sees (a subclass sets it)
         self.score_softcap, self.sink = 0.0, False      # (a subclass may bend the scores and add a sink to the softmax)
+        self.wide_weights = False      # True: the tensor-core kernel keeps the softmax weights to float32 precision (a subclass sets it)
         self.w_q_weight = self.w_k_weight = self.w_v_weight = self.w_output_weight = None
         self.w_qkv = None
         self._tc_tokens = {}     # cache shape -> tokens per tile of the tcgen05 kernel (0: not applicable)
@@ -112,6 +113,9 @@ class PagedAttention(Mixer):
         generic path, which has none)."""
         if not ops.attention_flash_supported(self.dtype, self.D):
             return None
+        return self._tensor_core_plans(ctx, cache)
+
+    def _tensor_core_plans(self, ctx, cache):
         Hq, Hkv, D = self.Hq, self.Hkv, self.D
         shape_key = (cache.page_size, cache.page_stride, cache.plane.dtype, cache.plane.dim())
         tc_tokens = self._tc_tokens.get(shape_key)
@@ -135,12 +139,13 @@ class PagedAttention(Mixer):
                 ops.set_work(ops.attention_work(ctx, Hq, Hkv, D, self.window, qkv.element_size()))
             if plan.kind == "tc":
                 ops.attention_tc(qkv, out, cache.plane, cache.page_stride, cache.page_size, table, ctx.q_start, ctx.pos0,
-                                 plan.work, plan.n_work, part_o, part_ml, Hq, Hkv, D, self.scale, self.window, ctx.err)
+                                 plan.work, plan.n_work, part_o, part_ml, Hq, Hkv, D, self.scale, self.window, ctx.err,
+                                 wide_weights=self.wide_weights)
             else:
                 ops.attention_flash(qkv, out, cache.plane, cache.page_stride, cache.page_size, table, ctx.q_start,
                                     ctx.pos0, plan.work, plan.n_work, part_o, part_ml, Hq, Hkv, D, self.scale,
                                     self.window, plan.bm, ctx.err, plan.cta_items, plan.n_ctas,
-                                    trigger_early=ctx.n_tokens <= EARLY_TRIGGER_MAX_TOKENS)
+                                    trigger_early=ctx.n_tokens <= EARLY_TRIGGER_MAX_TOKENS, wide_weights=self.wide_weights)
             if plan.n_comb:
                 ops.attention_combine(out, part_o, part_ml, ctx.q_start, ctx.req_of_token, plan.req_tile0,
                                       plan.tile_info, plan.comb_tokens, plan.n_comb, Hq, Hkv, D, plan.bm, plan.comb_warps)

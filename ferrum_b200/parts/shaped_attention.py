@@ -33,8 +33,10 @@ What a configuration may switch on, each with its constants as parameters:
                  must agree on kv heads x vdim.
 
 Scores, softmax weights, the weighted sum, rotations, the unit norm and the gate are float32 whatever
-the compute type (the CUDA-core attention kernel; keys, values and queries are stored in the compute
-type).  One product makes [q | k | v | gate logits] as float32 rows, `qkv_shape` shapes the heads
+the compute type (keys, values and queries are stored in the compute type).  The CUDA-core attention kernel does all of
+this.  With `wide_weights` a mixer whose heads need nothing between the two products but a causal mask or a window, and
+nothing after them, runs on the tensor cores where the head sizes allow it (`on_tensor_cores`): float32 scores and sums,
+and softmax weights that go into the second product as a 16-bit head and a 16-bit remainder.  One product makes [q | k | v | gate logits] as float32 rows, `qkv_shape` shapes the heads
 and writes the cache, the attention kernel leaves float32 results, `attention_finish` turns them back,
 gates them and rounds once for the output projection.  The reference's attention has none of these
 (crates/model/src/llama.rs:185-257).
@@ -50,12 +52,12 @@ from .linear import RESIDUAL, STORE_F32, linear, linear_deferred
 
 
 class ShapedAttention(PagedAttention):
-    graph_safe = True       # the CUDA-core attention kernel reads no work lists
+    graph_safe = True       # the CUDA-core attention kernel reads no work lists; the tensor-core one runs for groups of at most 16
 
     def __init__(self, width, n_head, n_head_kv, dim, vdim, dtype, scale, eps=1e-6, window=0, rotary=None, unit_norm=False,
                  value_rotary=None, distance_penalty=False, gate=False, mask="window", qkv_bias=False, qk_norm=False,
                  query_temperature=None, linear_bias=None, value_mix=None, value_mix_key="v_first", value_from_key=False,
-                 score_softcap=0.0, sink=False, keep_first=0):
+                 score_softcap=0.0, sink=False, keep_first=0, wide_weights=False):
         super().__init__(width, n_head, n_head_kv, max(int(dim), int(vdim)), rotary, dtype, window=window, scale=scale)
         self.keep_first = int(keep_first) if self.window > 0 else 0
         self.score_softcap, self.sink = float(score_softcap or 0.0), bool(sink)
@@ -92,6 +94,15 @@ class ShapedAttention(PagedAttention):
             raise ValueError("the value rotation covers all of a value head")
         self.w_r1 = self.w_r2 = self.w_g_weight = None
         self.w_in = None
+        self.wide_weights = bool(wide_weights)
+        bent = (self.has_penalty or self.linear_bias is not None or self.score_softcap > 0.0 or self.sink or self.chunked or self.keep_first
+                or self.has_gate or value_rotary is not None)
+        self.tensor_cores_fit = self.wide_weights and not bent and self.D == self.Dv and n_head // n_head_kv <= 16
+
+    def on_tensor_cores(self):
+        """Whether the attention itself runs on the tensor cores: heads of 64 or 128 (values at least as long as keys), 16-bit
+        storage, at most 16 query heads per KV head."""
+        return self.tensor_cores_fit and ops.attention_flash_supported(self.dtype, self.D)
 
     def param_specs(self):
         E = self.width
@@ -132,7 +143,7 @@ class ShapedAttention(PagedAttention):
         return CacheNeed(paged=PagedKVNeed(self.Hkv, self.D, self.window, keep_first=self.keep_first))
 
     def plan(self, ctx, cache):
-        return None
+        return self._tensor_core_plans(ctx, cache) if self.on_tensor_cores() else None
 
     @property
     def heads_width(self):
@@ -164,7 +175,9 @@ class ShapedAttention(PagedAttention):
                       k_norm=self.w_k_norm_weight if self.qk_norm else None, q_temp=self.q_temp, value_mix=mix,
                       whole_norm=self.whole_norm, value_from_key=self.value_from_key)
         penalty = (self.w_r1, self.w_r2) if self.has_penalty else ((self.slopes, None) if self.slopes is not None else None)
-        if Dp == Dv and vrot is None and not self.has_gate:
+        if scale == 1.0 and self.on_tensor_cores():
+            self._flash(q, out, ctx, cache, table)
+        elif Dp == Dv and vrot is None and not self.has_gate:
             # nothing is left to do to the heads' results: the attention kernel rounds its float32 sums once into `out`
             self._generic(q, out, ctx, cache, table, penalty, out_scale=scale)
         else:

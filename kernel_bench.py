@@ -5,7 +5,7 @@ peaks.  This is the small case that `ncu` captures are taken on.
 
     python kernel_bench.py attn_decode [--batch 8] [--context 8192] [--layers 4]
     python kernel_bench.py attn_prefill [--tokens 2048]
-    python kernel_bench.py gemm --tokens 8 --n 6144 --k 4096 [--epilogue store|residual|swiglu] [--copies 8]
+    python kernel_bench.py gemm --tokens 8 --n 6144 --k 4096 [--epilogue store|residual|swiglu|relu2] [--copies 8]
     python kernel_bench.py gemm|attn_decode|attn_prefill ... --dtype fp32    (the CUDA-core kernels of the 32-bit path)
     python kernel_bench.py latent_decode|latent_prefill [--hq 16] [--kv-rank 512] [--rot-dim 64] [--window W] [--cuda-cores]
     python kernel_bench.py head_linear --tokens 8 --hq 16 --n 512 --k 128
@@ -13,8 +13,10 @@ peaks.  This is the small case that `ncu` captures are taken on.
     python kernel_bench.py ssm --tokens 2048 [--batch 1] [--hq 64] [--head-dim 64] [--state 128]   (the state-space mixer's kernels)
     python kernel_bench.py delta|memory --tokens 2048 [--batch 1] [--hq 16] [--head-dim 128]   (the walks of the gated delta rule and of the matrix memory)
     python kernel_bench.py cdecay --tokens 2048 [--batch 1] [--hq 16] [--head-dim 128] [--bonus] [--segment L]   (the walk with a decay per key channel)
-    python kernel_bench.py moe --tokens 4096 --n 2816 --k 2048 [--experts 8] [--epilogue store|swiglu] [--mma-sync] [--cuda-cores]   (grouped product of a routed feed-forward)
+    python kernel_bench.py moe --tokens 4096 --n 2816 --k 2048 [--experts 8] [--epilogue store|swiglu|relu2] [--mma-sync] [--cuda-cores]   (grouped product of a routed feed-forward)
     python kernel_bench.py streams --tokens 2048 --k 2048 [--streams 4]   (write, read and norm over the residual streams)
+    python kernel_bench.py attn_*|latent_* ... --wide   (the tensor-core kernels with softmax weights kept to float32 precision)
+    python kernel_bench.py dyn_tanh --tokens 2048 --k 2048 [--top 2]   (the dynamic-tanh norm; --top: with the sum of that many expert rows)
     python kernel_bench.py rmsnorm|rope --tokens 8
     python kernel_bench.py step --tokens 2048 [--layers 2] [--dtype bf16|fp16|fp32]   (one prompt portion through the model)
     FERRUM_KERNEL_TRACE=1 python kernel_bench.py timeline [--batch 8] [--context 8192] [--layers 4]
@@ -39,7 +41,7 @@ sys.path.insert(0, ROOT)
 
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("kernel", choices=["attn_decode", "attn_prefill", "latent_decode", "latent_prefill", "head_linear", "gemm", "moe", "streams", "rmsnorm",
+    ap.add_argument("kernel", choices=["attn_decode", "attn_prefill", "latent_decode", "latent_prefill", "head_linear", "gemm", "moe", "streams", "rmsnorm", "dyn_tanh",
                                        "rope", "ssm", "delta", "memory", "cdecay", "step", "timeline"])
     ap.add_argument("--bonus", action="store_true", help="cdecay: the read-out before the write, with a bonus for the current token")
     ap.add_argument("--segment", type=int, default=-1, help="cdecay: tokens per segment (0: one piece; -1: the library's choice)")
@@ -59,7 +61,9 @@ def main():
     ap.add_argument("--tokens", type=int, default=8)
     ap.add_argument("--n", type=int, default=6144)
     ap.add_argument("--k", type=int, default=4096)
-    ap.add_argument("--epilogue", default="store", choices=["store", "residual", "swiglu"])
+    ap.add_argument("--epilogue", default="store", choices=["store", "residual", "swiglu", "relu2"])
+    ap.add_argument("--wide", action="store_true", help="attn_*, latent_*: softmax weights kept to float32 precision on the tensor cores")
+    ap.add_argument("--top", type=int, default=0, help="dyn_tanh: expert rows per token whose sum is made on the way")
     ap.add_argument("--ctas", type=int, default=0, help="gemm: CTAs of the grid (0 = one per SM)")
     ap.add_argument("--copies", type=int, default=8, help="distinct weight/cache copies cycled through, to defeat L2")
     ap.add_argument("--layers", type=int, default=4, help="cache planes cycled through (attention)")
@@ -118,6 +122,7 @@ def main():
         q = torch.randn(T, Hq * D, device=dev, generator=gen).to(td)
         out = torch.empty(T, Hq * D, device=dev, dtype=td)
         att = PagedAttention(Hq * D, Hq, Hkv, D, None, td)
+        att.wide_weights = args.wide
 
         class Cache:
             pass
@@ -220,7 +225,8 @@ def main():
             slots = longest // split + 2
             part = torch.empty(T * Hq * slots * (Rk + 2), device=dev)
         runs = [lambda pl=pl: ops.attention_latent(qf, out, gate, T, ctx, table, pl, pl.stride(0), ps, Hq, Dk, Rk, Dk ** -0.5, args.window,
-                                                   decode, part=part, split_slots=slots, tensor_cores=False if args.cuda_cores else None)
+                                                   decode, part=part, split_slots=slots, tensor_cores=False if args.cuda_cores else None,
+                                                   wide_weights=args.wide)
                 for pl in planes]
         keys, pairs = ops.visible_keys(ctx, args.window)
         work = {"bytes": keys * Dk * esize + T * Hq * (Dk + Rk) * esize, "flops": 2.0 * pairs * Hq * (Dk + Rk),
@@ -247,7 +253,7 @@ def main():
             epi = ops.TC_RESIDUAL
         else:
             o = torch.empty(M, N * (2 if dual and args.dtype == "fp32" else 1), device=dev, dtype=td)
-            epi = ops.TC_SWIGLU if dual else ops.TC_STORE_BF16
+            epi = ops.TC_SWIGLU if dual else (ops.TC_RELU2 if args.epilogue == "relu2" else ops.TC_STORE_BF16)
         if args.dtype == "fp32":     # the CUDA-core product (gate and up as one product of 2N rows; the activation is a kernel of its own)
             gepi = ops.EPI_RESIDUAL if args.epilogue == "residual" else ops.EPI_STORE
             runs = [lambda w=w: ops.gemm_generic(x, w, o, gepi) for w in weights]
@@ -263,17 +269,17 @@ def main():
     elif args.kernel == "moe":
         # --tokens sorted rows spread evenly over the experts (the last takes the remainder); swiglu: gate and up rows and the activation
         R, N, K, X = args.tokens, args.n, args.k, args.experts
-        glu = args.epilogue == "swiglu"
+        glu, unit = args.epilogue == "swiglu", args.epilogue == "relu2"
         share = [R // X] * X
         share[-1] += R - sum(share)
         counts = torch.tensor(share, dtype=torch.int32, device=dev)
         a = torch.randn(R, K, device=dev, generator=gen).to(td)
         weights = [torch.randn(X, N * (2 if glu else 1), K, device=dev, generator=gen).mul_(0.02).to(td) for _ in range(args.copies)]
-        o = torch.empty(R, N, device=dev, dtype=td if glu else torch.float32)
+        o = torch.empty(R, N, device=dev, dtype=td if glu or unit else torch.float32)
         ops.set_moe_cuda_cores(args.cuda_cores)
         ops.set_moe_tcgen05(not args.mma_sync)
         err = torch.zeros(1, dtype=torch.int32, device=dev)
-        runs = [lambda w=w: ops.moe_gemm(a, w, counts, R, o, N, glu="silu" if glu else None, err=err) for w in weights]
+        runs = [lambda w=w: ops.moe_gemm(a, w, counts, R, o, N, glu="silu" if glu else None, err=err, act="relu2" if unit else None) for w in weights]
         work = {"bytes": weights[0].numel() * esize + R * K * esize + o.numel() * o.element_size(),
                 "flops": 2.0 * R * N * K * (2 if glu else 1), "bound": "hbm" if R <= 32 * X else "tensor"}
     elif args.kernel == "streams":
@@ -285,6 +291,17 @@ def main():
         o = torch.empty(T, E, device=dev, dtype=td)
         runs = [lambda X=X: ops.hyper_step(X, S, E, T, write=ops.StreamWrite(mix, ow, y=y), in_w=iw, norm_w=w, eps=1e-6, out=o) for X in Xs]
         work = {"bytes": T * E * (8 * S + 4 + esize), "flops": 0.0, "bound": "hbm"}
+    elif args.kernel == "dyn_tanh":
+        T, E, top = args.tokens, args.k, args.top
+        xs = [torch.randn(T, E, device=dev, generator=gen) for _ in range(args.copies)]
+        w, b, alpha = torch.ones(E, device=dev), torch.zeros(E, device=dev), torch.full((1,), 0.5, device=dev)
+        o = torch.empty(T, E, device=dev, dtype=td)
+        ex = None
+        if top:
+            row_of = torch.randperm(T * top, device=dev).int()
+            ex = ops.ExpertSum(torch.randn(T * top, E, device=dev, generator=gen) * 0.01, row_of, top, torch.rand(T * top, device=dev))
+        runs = [lambda x=x: ops.dyn_tanh(x, alpha, w, b, o, experts=ex) for x in xs]
+        work = {"bytes": T * E * (4 + esize + (4 * top + 4 if top else 0)), "flops": 0.0, "bound": "hbm"}
     elif args.kernel == "rmsnorm":
         T, E = args.tokens, args.k
         x = torch.randn(T, E, device=dev, generator=gen)

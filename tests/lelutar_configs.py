@@ -8,6 +8,8 @@ B: everything a multiple of 8, so that 16-bit runs take the tensor-core products
 C: the smallest of everything: one head, keys of two, a latent of one, one expert in one group, no table of pairs.
 D: many experts in groups of one, negative scales, values above the keys' size, an unrotated attention, a mixture without
 groups, a scale of the embedding below one.
+E: attention heads of the sizes that the tensor-core attention takes (values as long as the keys, and longer), in a model
+without experts but for one layer, so that long requests compare row by row in 16 bits too.
 """
 import os
 
@@ -60,7 +62,21 @@ LELUTAR_D = {
          "mlp": {"kind": "moe", "expert": {"ff": 16}, "router": {"experts": 7, "top": 2}}},
     ],
 }
-LELUTAR = {"A": (LELUTAR_A, 3), "B": (LELUTAR_B, 4), "C": (LELUTAR_C, 5), "D": (LELUTAR_D, 6)}
+_ROT_E = {"base": 4000.0, "dims": 64, "scaling": {"factor": 6.0, "original": 96, "fast": 12.0, "slow": 1.0}}
+LELUTAR_E = {
+    "architecture": "Lelutar", "vocab": 144, "width": 96, "norm": {"eps": 1e-5}, "logit_scale": 0.9,
+    "embedding": {"scale": 2.0, "bigram": {"buckets": 77, "mul_prev": 13, "mul_cur": 29}},
+    "layers": [
+        {"type": "attention", "mixer": {"heads": 8, "kv_heads": 2, "dim": 64, "vdim": 64, "scale": 0.12, "rot": _ROT_E}, "mlp": {"kind": "dense", "ff": 120}},
+        {"type": "attention", "mixer": {"heads": 6, "kv_heads": 1, "dim": 40, "vdim": 128, "scale": 0.16, "rot": {"base": 100.0, "dims": 24}}, "mlp": None},
+        {"type": "latent_attention_2", "mixer": {"heads": 3, "dim": 16, "rot_dim": 16, "vdim": 24, "kv_rank": 32, "q_rank": 40, "scale": 0.25,
+                                                 "rot": {"base": 500.0, "dims": 16}},
+         "mlp": {"kind": "moe", "expert": {"ff": 32}, "router": {"experts": 6, "top": 2, "groups": {"count": 2, "keep": 1}}}},
+        {"type": "attention", "mixer": {"heads": 8, "kv_heads": 2, "dim": 64, "vdim": 64, "scale": 0.12, "rot": _ROT_E}, "mlp": {"kind": "dense", "ff": 120},
+         "weights_of": 0},
+    ],
+}
+LELUTAR = {"A": (LELUTAR_A, 3), "B": (LELUTAR_B, 4), "C": (LELUTAR_C, 5), "D": (LELUTAR_D, 6), "E": (LELUTAR_E, 7)}
 
 
 def write_model(cfg, folder, seed, std=0.12):

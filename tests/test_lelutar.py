@@ -8,7 +8,7 @@ import pytest
 import torch
 
 import plain_lelutar as P
-from lelutar_configs import LELUTAR_A, LELUTAR_B, LELUTAR_C, LELUTAR_D, write_model
+from lelutar_configs import LELUTAR_A, LELUTAR_B, LELUTAR_C, LELUTAR_D, LELUTAR_E, write_model
 
 from ferrum_b200.config import registry
 from ferrum_b200.config.lelutar import AttentionSpec, BigramSpec, LatentSpec, LelutarConfig
@@ -74,7 +74,7 @@ def build(d, dtype=torch.float32, **kw):
     return arch.build(arch.read_config(d), dtype, "cpu", **kw), arch
 
 
-@pytest.mark.parametrize("d", [LELUTAR_A, LELUTAR_B, LELUTAR_C, LELUTAR_D])
+@pytest.mark.parametrize("d", [LELUTAR_A, LELUTAR_B, LELUTAR_C, LELUTAR_D, LELUTAR_E])
 def test_tensor_names_cover_the_model_and_the_file(tmp_path, d):
     """The map from file names hits every tensor that the parts declare, once; a written file loads, and a missing,
     an unknown and a misshapen tensor are named in one error."""

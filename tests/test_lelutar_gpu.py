@@ -330,6 +330,71 @@ def test_wide_weights_keep_float32_precision(cuda, H, R, Rr):
     assert errs[True] < 2e-5 and errs[False] > 5 * errs[True], errs
 
 
+def plain_heads(q, k, v, pos, scale):
+    """q [n, H, D], k and v [keys, G, D] float64: causal grouped-query attention of queries at `pos`."""
+    G = k.shape[1]
+    out = torch.zeros_like(q)
+    for t, p in enumerate(pos):
+        for h in range(q.shape[1]):
+            g = h // (q.shape[1] // G)
+            out[t, h] = torch.softmax(k[:p + 1, g] @ q[t, h] * scale, dim=0) @ v[:p + 1, g]
+    return out
+
+
+@pytest.mark.parametrize("dtype", ["bfloat16", "float16"])
+@pytest.mark.parametrize("H,G,D,page", [(8, 2, 64, 16), (4, 4, 128, 8), (16, 1, 64, 32), (6, 2, 128, 16)])
+def test_grouped_attention_with_wide_weights(cuda, dtype, H, G, D, page):
+    """Values of +-64 around a small signal: what the weights lose to rounding shows in the result unless they keep their
+    precision.  Prompt portions, one token over a range that is cut among CTAs, the first tokens; a far dominant key."""
+    from ferrum_b200.cache.storage import LayerCache
+    from ferrum_b200.parts import ShapedAttention
+    td, n_keys, rng = TD[dtype], 620, np.random.default_rng(D)
+    n_pages = -(-n_keys // page)
+    order = rng.permutation(n_pages + 4)[:n_pages]
+    k = rng.standard_normal((n_keys, G, D)) * 0.4
+    v = rng.standard_normal((n_keys, G, D))
+    v[0::2] += 64.0
+    v[1::2] -= 64.0
+    kt, vt = torch.tensor(k, device="cuda").to(td), torch.tensor(v, device="cuda").to(td)
+    plane = torch.zeros(n_pages + 4, 2, G, page, D, device="cuda", dtype=td)
+    for lp in range(n_pages):
+        n = min(page, n_keys - lp * page)
+        plane[order[lp], 0, :, :n] = kt[lp * page:lp * page + n].transpose(0, 1)
+        plane[order[lp], 1, :, :n] = vt[lp * page:lp * page + n].transpose(0, 1)
+    cache = LayerCache(group=0, plane=plane, page_stride=plane.stride(0), page_size=page, writes=True, state=None)
+    mixer = ShapedAttention(32, H, G, D, D, td, 0.2, wide_weights=True)
+    assert mixer.on_tensor_cores()
+
+    def run(q, pos0, n):
+        ctx = make_ctx([(pos0, n)], widths=[[[int(p) for p in order]]])
+        out = torch.full((n, H * D), float("nan"), device="cuda", dtype=td)
+        mixer._flash(q, out, ctx, cache, ctx.block_tables[0])
+        assert ctx.err.item() == 0
+        return out.double().view(n, H, D)
+    unit = 2.0 ** (-8 if dtype == "bfloat16" else -11)            # (a result's own rounding is half of this)
+    for pos0, n in ((n_keys - 170, 170), (n_keys - 70, 70), (n_keys - 1, 1), (100, 2), (0, 5), (0, 140)):
+        qt = torch.tensor(rng.standard_normal((n, H * D)) * 0.5, device="cuda").to(td)
+        ref = plain_heads(qt.double().view(n, H, D), kt.double(), vt.double(), list(range(pos0, pos0 + n)), 0.2)
+        errs = []
+        for mixer.wide_weights in (True, False):
+            errs.append(((run(qt, pos0, n) - ref).abs() / ref.abs().clamp_min(1.0)).max().item())
+        assert errs[0] < unit + 2e-3, (pos0, n, errs)
+        if n in (70, 170):
+            assert errs[1] > 2.0 * errs[0], errs
+    mixer.wide_weights = True
+    hot = page * 7 - 1                       # a page's last row, far back
+    kt[hot] *= 8.0
+    plane[order[hot // page], 0, :, hot % page] = kt[hot]
+    for pos0, n in ((n_keys - 70, 70), (n_keys - 1, 1), (hot - 1, 3), (hot - 100, 300)):
+        if pos0 < 0:
+            continue
+        qt = (kt[hot].double().repeat_interleave(H // G, dim=0).reshape(1, H * D).repeat(n, 1) * 2.0).to(td)
+        got = run(qt, pos0, n)
+        for i in range(n):
+            near = (got[i] - vt[hot].double().repeat_interleave(H // G, dim=0)).abs().max()
+            assert (near < 1.0) == (pos0 + i >= hot), (pos0, i)
+
+
 # ================================================================= mixers alone, whole and in portions
 CUTS = ([61], [20, 1, 1, 2, 30, 7], [2] * 30 + [1], [1] * 61)
 
@@ -359,14 +424,17 @@ YARN = {"factor": 4.0, "original": 40, "fast": 8.0, "slow": 1.0}
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("H,G,D,Dv,rot", [(6, 2, 10, 14, {"base": 60.0, "dims": 6, "scaling": YARN}), (4, 4, 32, 16, {"base": 500.0, "dims": 32, "scaling": YARN}),
                                           (3, 1, 8, 24, {"base": 20.0, "dims": 8}), (2, 1, 2, 1, {"base": 9.0, "dims": 2, "scaling": YARN}), (10, 2, 6, 6, None),
-                                          (8, 1, 64, 96, {"base": 10000.0, "dims": 64, "scaling": YARN}), (2, 2, 128, 128, {"base": 100.0, "dims": 40})])
+                                          (8, 1, 64, 96, {"base": 10000.0, "dims": 64, "scaling": YARN}), (2, 2, 128, 128, {"base": 100.0, "dims": 40}),
+                                          (8, 1, 40, 64, {"base": 500.0, "dims": 24, "scaling": YARN}), (16, 1, 128, 128, None), (17, 1, 64, 64, None)])
 def test_rotating_attention_alone(cuda, dtype, H, G, D, Dv, rot):
     from ferrum_b200.parts import ShapedAttention
     td, E = TD[dtype], 40
-    mixer = ShapedAttention(E, H, G, D, Dv, td, 0.45, rotary=table_of(rot, D), qkv_bias=True)
+    scale = 0.45 if D < 64 else 0.1
+    mixer = ShapedAttention(E, H, G, D, Dv, td, scale, rotary=table_of(rot, D), qkv_bias=True, wide_weights=True)
+    assert mixer.on_tensor_cores() == (dtype == "bfloat16" and max(D, Dv) in (64, 128) and Dv >= D and H // G <= 16)
     w = fill_part(mixer, 9, td, "p.")
     x = inputs(61, E, td)
-    m = {"heads": H, "kv_heads": G, "dim": D, "vdim": Dv, "scale": 0.45, "rot": rot}
+    m = {"heads": H, "kv_heads": G, "dim": D, "vdim": Dv, "scale": scale, "rot": rot}
     ref = P.attention(x.double().cpu(), w, "p.", m, 1e-5, rounding_of(dtype))
     check_mixer(mixer, ref, x, td, dtype)
     if rot:                   # what a half-split pairing, or a magnitude that is left out, would give is something else
@@ -555,10 +623,10 @@ def test_ungated_experts_alone(cuda, dtype, E, F, n_exp, top, groups, T):
 
 
 # ================================================================= whole models, every way of cutting the work
-CASES = [(n, d) for n in ("A", "B") for d in ("float32", "bfloat16")]
+CASES = [(n, d) for n in ("A", "B") for d in ("float32", "bfloat16")] + [("E", "bfloat16")]
 
 
-@pytest.mark.parametrize("name,dtype", CASES + [("C", "float32"), ("C", "bfloat16"), ("D", "float32"), ("D", "bfloat16")])
+@pytest.mark.parametrize("name,dtype", CASES + [("C", "float32"), ("C", "bfloat16"), ("D", "float32"), ("D", "bfloat16"), ("E", "float32")])
 def test_whole_prompt_and_first_tokens(cuda, folders, name, dtype):
     toks = tokens_for(name, 140, 10, folders)
     r = Replay(session(folders[name], dtype, 160))
@@ -571,7 +639,7 @@ def test_whole_prompt_and_first_tokens(cuda, folders, name, dtype):
     close(r.logits("b", 4), plain(folders[name], dtype, toks[:4]), dtype, f"{name} first tokens")
 
 
-@pytest.mark.parametrize("name", ["A", "B", "C", "D"])
+@pytest.mark.parametrize("name", ["A", "B", "C", "D", "E"])
 def test_residual_rows_after_every_layer_run(cuda, folders, name):
     toks = tokens_for(name, 25, 11, folders)
     cfg, w = P.load(folders[name])
@@ -689,6 +757,30 @@ def test_a_long_prompt_and_a_far_token(cuda, folders):
         assert d[5] > 1e-3 and d[-20:].min() > 1e-5 and d[:5].max() < 1e-5
 
 
+@pytest.mark.parametrize("dtype", ["bfloat16", "float16"])
+def test_long_requests_on_the_tensor_core_attention(cuda, folders, dtype):
+    """Three requests of hundreds of tokens, portions of all sizes beside single tokens in one batch: rows go to every kernel of the
+    tensor-core attention (the work lists' three classes, key ranges cut among CTAs) in the same step."""
+    lens = {"a": 400, "b": 333, "c": 290}
+    toks = {k: tokens_for("E", n, 70 + i, folders) for i, (k, n) in enumerate(lens.items())}
+    s = session(folders["E"], dtype, 1200, page_size=16)
+    assert all(b.mixer.on_tensor_cores() for b in s.model.blocks[:2])
+    r, at = Replay(s), {k: 0 for k in lens}
+    sizes = {"a": [150, 1, 3, 200, 1, 40], "b": [1, 2, 17, 130, 1, 180], "c": [64, 190, 1, 1, 30, 2]}
+    step = 0
+    while any(at[k] < lens[k] for k in lens):
+        entries = []
+        for k in lens:
+            n = min(sizes[k][step % 6], lens[k] - at[k])
+            if n:
+                entries.append((k, toks[k][at[k]:at[k] + n], "all"))
+                at[k] += n
+        r.step(entries)
+        step += 1
+    for k in lens:
+        close(r.logits(k, lens[k]), plain(folders["E"], dtype, toks[k]), dtype, f"E long {k}")
+
+
 def plain_generate(cfg, w, prompt, n, rd=None):
     seq = list(prompt)
     for _ in range(n):
@@ -696,7 +788,7 @@ def plain_generate(cfg, w, prompt, n, rd=None):
     return seq[len(prompt):]
 
 
-@pytest.mark.parametrize("name,dtype", [("A", "float32"), ("B", "float32"), ("B", "bfloat16"), ("D", "float32")])
+@pytest.mark.parametrize("name,dtype", [("A", "float32"), ("B", "float32"), ("B", "bfloat16"), ("D", "float32"), ("E", "bfloat16")])
 def test_greedy_generation_through_the_engine(cuda, folders, name, dtype):
     """Engine.generate (scheduler, sampler, chunked prompts, several requests, steps planned ahead whose tokens never leave the
     device) against the plain implementation; in bfloat16 a token may differ only at a near-tie of the plain logits."""
