@@ -672,9 +672,9 @@ def group_configs(size, layers, vocab=32000, window=4096):
     s = GROUP_SIZES[size]
     yarn = {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}
     att = {"type": "attention", "mixer": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["vdim"], "scale": s["dim"] ** -0.5,
-                                          "rot": {"base": 50000.0, "dims": s["dim"], "scaling": yarn}}}
+                                          "rot": {"base": 100000.0, "dims": s["dim"], "scaling": yarn}}}
     lat = {"heads": s["heads"], "dim": s["dim"], "vdim": s["vdim"], "kv_rank": s["kv_rank"], "q_rank": s["q_rank"], "scale": s["dim"] ** -0.5}
-    turned = dict(lat, rot_dim=s["rot_dim"], scale=(s["dim"] + s["rot_dim"]) ** -0.5, rot={"base": 50000.0, "dims": s["rot_dim"], "scaling": yarn})
+    turned = dict(lat, rot_dim=s["rot_dim"], scale=(s["dim"] + s["rot_dim"]) ** -0.5, rot={"base": 100000.0, "dims": s["rot_dim"], "scaling": yarn})
     dense = {"kind": "dense", "ff": s["ff"]}
     moe = {"kind": "moe", "expert": {"ff": s["expert_ff"]},
            "router": {"experts": s["experts"], "top": s["top"], "groups": {"count": s["groups"], "keep": s["keep"]}}}

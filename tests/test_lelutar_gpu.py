@@ -424,7 +424,7 @@ YARN = {"factor": 4.0, "original": 40, "fast": 8.0, "slow": 1.0}
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("H,G,D,Dv,rot", [(6, 2, 10, 14, {"base": 60.0, "dims": 6, "scaling": YARN}), (4, 4, 32, 16, {"base": 500.0, "dims": 32, "scaling": YARN}),
                                           (3, 1, 8, 24, {"base": 20.0, "dims": 8}), (2, 1, 2, 1, {"base": 9.0, "dims": 2, "scaling": YARN}), (10, 2, 6, 6, None),
-                                          (8, 1, 64, 96, {"base": 10000.0, "dims": 64, "scaling": YARN}), (2, 2, 128, 128, {"base": 100.0, "dims": 40}),
+                                          (7, 1, 64, 96, {"base": 10000.0, "dims": 64, "scaling": YARN}), (2, 2, 128, 128, {"base": 100.0, "dims": 40}),
                                           (8, 1, 40, 64, {"base": 500.0, "dims": 24, "scaling": YARN}), (16, 1, 128, 128, None), (17, 1, 64, 64, None)])
 def test_rotating_attention_alone(cuda, dtype, H, G, D, Dv, rot):
     from ferrum_b200.parts import ShapedAttention
@@ -555,7 +555,7 @@ def test_group_choice_by_hand(cuda, T):
     assert route(2, (3, 1), zero, lg=tiny)[1][0] == [0.0, 0.0]
 
 
-@pytest.mark.parametrize("n_exp,top,groups", [(12, 2, (3, 2)), (64, 6, (8, 4)), (256, 8, (8, 4)), (256, 8, (64, 7)), (96, 5, (96, 40)), (40, 3, (5, 5)), (7, 7, (1, 1))])
+@pytest.mark.parametrize("n_exp,top,groups", [(12, 3, (4, 2)), (64, 6, (8, 4)), (256, 8, (8, 4)), (256, 8, (64, 7)), (96, 5, (96, 40)), (40, 3, (5, 5)), (7, 7, (1, 1))])
 def test_group_choice_against_the_plain_one(cuda, n_exp, top, groups):
     """Random scores with corrections of both signs; the two routing kernels (few and many tokens)."""
     from ferrum_b200.ops import lib as ops
